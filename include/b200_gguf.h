@@ -140,8 +140,9 @@ int b2_synchronize(b2_engine* e);
 #define B2_MIX_WINDOW_SCAN 1     /* sliding-window attention with a kept prefix (values = raw keys) beside a selective
                                     scan (Mamba); the two outputs are RMS-normed over the width and averaged */
 #define B2_MIX_MATRIX_MEMORY 2   /* mLSTM: per-head matrix memory with capped exponential gating */
-#define B2_MIX_LATENT_ATTN 3     /* sliding-window attention over one cached low-rank latent + one shared rotated key part
-                                    per token, per-head softmax sink, sigmoid output gate */
+#define B2_MIX_LATENT_ATTN 3     /* attention over one cached low-rank latent + one shared rotated key part per token (either may be
+                                    read from an earlier layer: kv_from), optionally a sliding window, queries through a latent of their
+                                    own (la_q_rank), a softmax sink per head, a sigmoid output gate (attn_flags) */
 #define B2_MIX_DELTA_RULE 4      /* gated delta rule: per-head matrix memory with per-row input-dependent decays, short
                                     causal convolutions on q / k / v */
 #define B2_MIX_SSD 5             /* Mamba-2 state-space recurrence: scalar decay per head, grouped B / C, gated group norm */
@@ -155,17 +156,23 @@ int b2_synchronize(b2_engine* e);
 #define B2_MIX_SINK_ATTN 8       /* the same softmax attention alone; what differs is chosen by attn_flags */
 #define B2_FF_RELU2 0            /* squared-ReLU block with biases (when n_ff > 0) */
 #define B2_FF_MOE 1              /* routed mixture of gated (SiLU) experts, n_ff = width of one expert */
-#define B2_FF_GLU 2              /* gated SiLU unit without biases: down(silu(gate x) * (up x)) */
+#define B2_FF_GLU 2              /* gated unit without biases: down(act(gate x) * (up x)), act = ff_act */
 #define B2_FF_PIECEWISE 3        /* down(act(up x)) without biases; act(z) = a z^2 + z / 2 for z > 0, b (exp(z) - 1 - z) + z / 2 otherwise,
                                     a = softplus(p), b = 1/2 + softplus(q) with (p, q) in tensor mlp.act */
+#define B2_ACT_SILU 0            /* ff_act: z * sigmoid(z) */
+#define B2_ACT_GELU_TANH 1       /* ff_act: z / 2 * (1 + tanh(sqrt(2 / pi) * (z + 0.044715 z^3))) */
 #define B2_EXPERT_SILU 0         /* expert: down(silu(gate x) * (up x)) */
 #define B2_EXPERT_CLAMPED 1      /* expert: g = min(gate x, limit), u = clamp(up x, -limit, limit); down(g * sigmoid(alpha g) * (u + 1)) */
 #define B2_ATTN_BIAS 1           /* attn_flags: q, k, v projections carry biases (tensors q.b, k.b, v.b) */
 #define B2_ATTN_UNIT_QK 2        /* after the rotation every head's q and k are divided by their RMS (no weight) */
 #define B2_ATTN_TALK 4           /* weight_h(i, j) <- sum_g talk[h][g] weight_g(i, j) after the softmax (tensor talk [H][H]) */
 #define B2_ATTN_HEAD_GATE 8      /* the sigmoid output gate is one number per head (tensor g [H][W]); else one per output entry */
+#define B2_ATTN_NO_GATE 16       /* latent attention: no output gate (no tensor g) */
+#define B2_ATTN_NO_SINK 32       /* latent attention: ordinary softmax (no tensor sink) */
+#define B2_ATTN_ROT_PAIRS 64     /* latent attention: entries 2i and 2i + 1 are rotated together; else i and i + rot_dims / 2 */
 #define B2_ROUTE_SOFTMAX_ALL 0   /* scores = softmax over all slots; an additive correction steers the choice only */
 #define B2_ROUTE_TOPK_SOFTMAX 1  /* biased logits choose; weights = softmax over the chosen logits */
+#define B2_ROUTE_SIGMOID 2       /* scores = sigmoid of each logit; the largest (+ correction, if any) are chosen */
 #define B2_BLOCK_POSTSUM_LN 0    /* x <- LayerNorm(alpha * x + f(x)) */
 #define B2_BLOCK_PRENORM_RMS 1   /* x <- x + m * f(RMSNorm(x) * (1 + w)); the embedding and the output are normed the same way */
 #define B2_BLOCK_OUTNORM_RMS 2   /* x <- x + RMSNorm_parts(f(x)) * w: the branch OUTPUT is normed, over norm_groups equal parts;
@@ -175,6 +182,8 @@ int b2_synchronize(b2_engine* e);
                                     (h + conv(h), tensors l<i>.canon1/2 [W][taps]); its output y goes back as
                                     x_t <- sum_s mix[s][t] x_s + out[t] y (tensors l<i>.hc1/2.in, .mix, .out; absent: plain residual).
                                     The output norm reads the sum of the copies. */
+#define B2_BLOCK_PARALLEL_LN 4   /* x <- x + (mixer(LN1(x)) + ff(LN2(x))), both of the same x; LN with weight and bias (tensors norm1,
+                                    norm1.b, ...); the output norm has the same form */
 typedef struct b2_layer_desc {
     int32_t mixer;            /* B2_MIX_* */
     int32_t n_ff;             /* width of the feed-forward block (of one expert for B2_FF_MOE); 0 = the layer has none */
@@ -211,6 +220,12 @@ typedef struct b2_layer_desc {
     int32_t moe_renorm;       /* != 0: the chosen scores are divided by their sum (+ 1e-20) */
     double moe_limit;         /* B2_EXPERT_CLAMPED */
     double moe_alpha;         /* B2_EXPERT_CLAMPED: slope inside the sigmoid */
+    int32_t ff_act;           /* B2_FF_GLU: B2_ACT_* */
+    int32_t moe_scale_input;  /* != 0: a choice's weight multiplies the expert's input; the outputs are added as they are */
+    int32_t la_q_rank;        /* latent attention: size of the normed query latent (tensors dq, dq.norm, uq); 0: queries come from the
+                                 input by one map (tensor q) */
+    int32_t kv_from;          /* latent attention: 1 + index of the earlier layer whose cached rows this one reads (it has no dkv of
+                                 its own); 0: its own */
 } b2_layer_desc;
 typedef struct b2_layered_config {
     int32_t n_layer, n_embd, n_vocab;
@@ -227,6 +242,9 @@ typedef struct b2_layered_config {
     int32_t tie_head;         /* != 0: the output map is the embedding table (no tensor "head") */
     int32_t n_streams;        /* B2_BLOCK_HYPER_RMS: copies of the residual stream (0 is read as 1) */
     int32_t canon_taps;       /* B2_BLOCK_HYPER_RMS: taps of the convolution on every sublayer's input (0: none) */
+    /* bigram embedding: the row (previous token * mul_prev + token * mul_cur) mod buckets of tensor "bigram" [buckets + 1] is added to
+     * the embedding row; a sequence's first token takes row `buckets`. 0 buckets: none. The factors are given mod buckets. */
+    int32_t bigram_buckets, bigram_mul_prev, bigram_mul_cur;
 } b2_layered_config;
 /* Then b2_upload_tensor for every tensor (BF16 / F32), b2_engine_finalize, b2_seq_set_blocks / b2_seq_begin (n_past must be
  * 0: recurrent state cannot be rewound; it zeroes the slot's state) as for any engine. */

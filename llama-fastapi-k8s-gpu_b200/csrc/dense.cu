@@ -26,7 +26,7 @@ struct DenseDev {
     float* y; int ldy;
     int T, N, K, epi;
     float scale, p0, p1;
-    const float* aux; int ldaux;
+    const float* aux; int ldaux, aux_ns;      // aux column of output column n: n * aux_ns
     long x_bs, w_bs, y_bs, aux_bs;
     int grouped;                   // 0 plain, 1 one pair per blockIdx.y, 2 tiles
     DenseGroups g;
@@ -60,18 +60,20 @@ __device__ __forceinline__ bool dense_tile(const DenseDev& a, int rows_per_cta, 
 __device__ __forceinline__ int x_row(const DenseDev& a, int t) { return (a.grouped && a.g.x_rows) ? a.g.x_rows[t] : t; }
 
 __device__ __forceinline__ float silu_act(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float gelu_tanh_act(float z) { return 0.5f * z * (1.f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z))); }
 // one output column
 __device__ __forceinline__ void epi_store(const DenseDev& a, float* y, const float* aux, int t, int n, float v) {
     if (a.epi == EPI_BIAS || a.epi == EPI_BIAS_RELU2) { if (a.bias) v += a.bias[n]; }
     if (a.epi == EPI_BIAS_RELU2) { v = fmaxf(v, 0.f); v = v * v; }
-    if (a.epi == EPI_MUL_SIGMOID) v *= 1.f / (1.f + expf(-aux[(size_t)t * a.ldaux + n]));
+    if (a.epi == EPI_MUL_SIGMOID) v *= 1.f / (1.f + expf(-aux[(size_t)t * a.ldaux + n * a.aux_ns]));
     if (a.epi == EPI_PIECEWISE) v = v > 0.f ? fmaf(a.p0 * v, v, 0.5f * v) : fmaf(a.p1, expm1f(v) - v, 0.5f * v);
     y[(size_t)t * a.ldy + n] = v * a.scale;
 }
-// two neighbouring columns n (even) and n + 1
-__device__ __forceinline__ void epi_store2(const DenseDev& a, float* y, const float* aux, int t, int n, float v0, float v1) {
-    if (a.epi == EPI_GLU_SILU) {
-        if (n + 1 < a.N) y[(size_t)t * a.ldy + (n >> 1)] = silu_act(v0) * v1 * a.scale;
+// two neighbouring columns n (even) and n + 1; rs: scales of the product rows (GLU epilogues) or null
+__device__ __forceinline__ void epi_store2(const DenseDev& a, float* y, const float* aux, const float* rs, int t, int n, float v0, float v1) {
+    if (rs) { v0 *= rs[t]; v1 *= rs[t]; }
+    if (a.epi == EPI_GLU_SILU || a.epi == EPI_GLU_GELU) {
+        if (n + 1 < a.N) y[(size_t)t * a.ldy + (n >> 1)] = (a.epi == EPI_GLU_SILU ? silu_act(v0) : gelu_tanh_act(v0)) * v1 * a.scale;
         return;
     }
     if (a.epi == EPI_GLU_CLAMP) {
@@ -101,7 +103,8 @@ __global__ void __launch_bounds__(256) dense_rows_kernel(DenseDev a) {
     const float* x; const TW* w; float* y; const float* aux; int t0, t1;
     if (!dense_tile<TW>(a, ROWS_MAX_T, x, w, y, aux, t0, t1)) return;
     const int T = a.grouped ? 1 : a.T;
-    if (a.grouped) { x += (size_t)x_row(a, t0) * ldx; y += (size_t)t0 * a.ldy; if (aux) aux += (size_t)t0 * a.ldaux; }
+    const float* rs = a.g.row_scale;
+    if (a.grouped) { x += (size_t)x_row(a, t0) * ldx; y += (size_t)t0 * a.ldy; if (aux) aux += (size_t)t0 * a.ldaux; if (rs) rs += t0; }
     const TW* rows[R];
 #pragma unroll
     for (int r = 0; r < R; r++) rows[r] = w + (size_t)min(n0 + r, N - 1) * K;      // past the end: the last row again, not stored
@@ -175,7 +178,7 @@ __global__ void __launch_bounds__(256) dense_rows_kernel(DenseDev a) {
         if (lane != 0) continue;
         if constexpr (R % 2 == 0) {
 #pragma unroll
-            for (int r = 0; r < R; r += 2) epi_store2(a, y, aux, t, n0 + r, v[r], v[r + 1]);
+            for (int r = 0; r < R; r += 2) epi_store2(a, y, aux, rs, t, n0 + r, v[r], v[r + 1]);
         } else {
             epi_store(a, y, aux, t, n0, v[0]);
         }
@@ -188,7 +191,7 @@ static cudaError_t launch_rows(const DenseDev& d, int batch, cudaStream_t s) {
     const unsigned gy = d.grouped ? d.T : 1, gz = d.grouped ? 1 : batch;       // grouped: one pair row per blockIdx.y
     const int N = d.N;
     if (d.grouped || d.T == 1) {
-        if (d.epi == EPI_GLU_SILU || d.epi == EPI_GLU_CLAMP) return launch_chain(dense_rows_kernel<TW, 1, 2>, dim3((N + 15) / 16, gy, gz), block, 0, s, d);
+        if (d.epi == EPI_GLU_SILU || d.epi == EPI_GLU_GELU || d.epi == EPI_GLU_CLAMP) return launch_chain(dense_rows_kernel<TW, 1, 2>, dim3((N + 15) / 16, gy, gz), block, 0, s, d);
         return launch_chain(dense_rows_kernel<TW, 1, 1>, dim3((N + 7) / 8, gy, gz), block, 0, s, d);
     }
     if (d.T == 2) return launch_chain(dense_rows_kernel<TW, 2, 2>, dim3((N + 15) / 16, gy, gz), block, 0, s, d);
@@ -209,6 +212,7 @@ __global__ void __launch_bounds__(256) dense_fma_kernel(DenseDev a) {
     const int N = a.N, K = a.K, ldx = a.ldx;
     const int n0 = blockIdx.x * BN;
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;      // thread tile: rows ty*4.., cols tx*4..
+    const float* rs = a.g.row_scale;
     float acc[4][4] = {};
     for (int k0 = 0; k0 < K; k0 += BK) {
         for (int i = threadIdx.x; i < BM * BK; i += 256) {
@@ -236,7 +240,7 @@ __global__ void __launch_bounds__(256) dense_fma_kernel(DenseDev a) {
         const int t = t0 + ty * 4 + i;
         if (t >= T) continue;
 #pragma unroll
-        for (int j = 0; j < 4; j += 2) epi_store2(a, y, aux, t, n0 + tx * 4 + j, acc[i][j], acc[i][j + 1]);
+        for (int j = 0; j < 4; j += 2) epi_store2(a, y, aux, rs, t, n0 + tx * 4 + j, acc[i][j], acc[i][j + 1]);
     }
 }
 
@@ -323,7 +327,7 @@ __global__ void __launch_bounds__(128) dense_mma_kernel(DenseDev a) {
 #pragma unroll
             for (int e = 0; e < 4; e += 2) {
                 const int t = t0 + wm + mi * 16 + g + (e >> 1) * 8;
-                if (t < T) epi_store2(a, y, aux, t, n0 + wn + ni * 8 + 2 * tq, acc[mi][ni][e], acc[mi][ni][e + 1]);
+                if (t < T) epi_store2(a, y, aux, a.g.row_scale, t, n0 + wn + ni * 8 + 2 * tq, acc[mi][ni][e], acc[mi][ni][e + 1]);
             }
 }
 
@@ -424,19 +428,19 @@ __global__ void __launch_bounds__(256, 2) dense_mma_big_kernel(const __nv_bfloat
 #pragma unroll
             for (int e = 0; e < 4; e += 2) {
                 const int t = t0 + wm + mi * 16 + g + (e >> 1) * 8;
-                if (t < T) epi_store2(a, y, aux, t, n0 + wn + ni * 8 + 2 * tq, acc[mi][ni][e], acc[mi][ni][e + 1]);
+                if (t < T) epi_store2(a, y, aux, a.g.row_scale, t, n0 + wn + ni * 8 + 2 * tq, acc[mi][ni][e], acc[mi][ni][e + 1]);
             }
 }
 
 cudaError_t dense_launch(const DenseArgs& a, cudaStream_t s) {
     if (a.T <= 0 || a.N <= 0 || a.K <= 0 || a.batch <= 0) return cudaErrorInvalidValue;
     if (a.w_type != T_BF16 && a.w_type != T_F32) return cudaErrorInvalidValue;
-    if ((a.epi == EPI_GLU_SILU || a.epi == EPI_GLU_CLAMP) && a.N % 2) return cudaErrorInvalidValue;
+    if ((a.epi == EPI_GLU_SILU || a.epi == EPI_GLU_GELU || a.epi == EPI_GLU_CLAMP) && a.N % 2) return cudaErrorInvalidValue;
     if (a.groups && a.batch != 1) return cudaErrorInvalidValue;
     const bool wb = a.w_type == T_BF16;
     DenseDev d = {};
     d.x = a.x; d.ldx = a.ldx; d.w = a.w; d.bias = a.bias; d.y = a.y; d.ldy = a.ldy; d.T = a.T; d.N = a.N; d.K = a.K; d.epi = a.epi;
-    d.scale = a.scale; d.p0 = a.p0; d.p1 = a.p1; d.aux = a.aux; d.ldaux = a.ldaux; d.x_bs = a.x_bs; d.w_bs = a.w_bs; d.y_bs = a.y_bs; d.aux_bs = a.aux_bs;
+    d.scale = a.scale; d.p0 = a.p0; d.p1 = a.p1; d.aux = a.aux; d.ldaux = a.ldaux; d.aux_ns = a.aux_one ? 0 : 1; d.x_bs = a.x_bs; d.w_bs = a.w_bs; d.y_bs = a.y_bs; d.aux_bs = a.aux_bs;
     if (a.groups) { d.g = *a.groups; d.grouped = a.groups->tile_group ? 2 : 1; }
     if (d.grouped == 1 || (!d.grouped && a.T <= ROWS_MAX_T)) return wb ? launch_rows<__nv_bfloat16>(d, a.batch, s) : launch_rows<float>(d, a.batch, s);
     // few output columns in 32-bit (router scores): the tiled kernel would run a handful of CTAs over the whole K; the

@@ -657,6 +657,7 @@ extern "C" int b2_seq_begin(b2_engine* e, int slot, int n_past, const int32_t* h
     if (n_uni) CK(cudaMemcpyAsync(s.uniforms, uni, sizeof(double) * n_uni, cudaMemcpyHostToDevice, e->stream));
     CK(cudaStreamSynchronize(e->stream));
     s.n_past = n_past;
+    s.last_token = -1;
     s.n_sampled = 0;
     return B2_OK;
 }

@@ -51,6 +51,7 @@ struct Slot {
     int n_decode_nodes = 0, n_pre_step_nodes = 0, n_pre_last_nodes = 0, n_fwd_nodes = 0;
     const float* logits_view = nullptr;   // where the latest logits of this slot are (own buffer, or a row of the batch output)
     int n_past = 0;                // host mirror of ints[1]
+    int last_token = -1;           // layer-list models: the token at position n_past - 1 (-1: none yet)
     int n_sampled = 0;             // host mirror of ints[3]
 };
 

@@ -62,7 +62,7 @@ __device__ __forceinline__ void hyper_token(const HyperDev& p, int t, float* hy_
                 for (int c = 0; c < j.top; c++) {
                     const int q = t * j.top + c, e = j.sel[q];
                     const float v = e < j.n_experts ? j.rows[(size_t)(j.pos ? j.pos[q] : q) * W + i] : j.h[base + i];
-                    y = fmaf(j.weight[q], v, y);
+                    y = fmaf(j.weight ? j.weight[q] : 1.f, v, y);
                 }
             }
             float nx[SM];

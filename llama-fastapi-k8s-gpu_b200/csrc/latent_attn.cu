@@ -2,8 +2,9 @@
 // low-rank latent) that all heads read; keys and values are linear maps of c per head. The key map is folded into the
 // query (the caller multiplies each head's unrotated query by W_uk,h^T), so a score is one dot product of the folded
 // query [rank + dr] with the cached row, and the softmax-weighted sum runs over the c parts; the value map is applied
-// afterwards to that sum. Sliding window, and a per-head sink term in the softmax denominator (it has no value).
-// Softmax, the norm of c and the rotation are 32-bit; only the cached rows may be bf16.
+// afterwards to that sum. Sliding window, and optionally a per-head sink term in the softmax denominator (it has no value).
+// A layer may read the rows that an earlier layer caches (ld_row is that layer's row length). Softmax, the norms of the
+// latents and the rotation are 32-bit; only the cached rows may be bf16.
 #include "kernels.h"
 #include "layered.h"
 #include "ptx.cuh"
@@ -22,13 +23,22 @@ __device__ __forceinline__ void row_store(void* pool, int f32, size_t i, float v
 __device__ __forceinline__ float row_load(const void* pool, int f32, size_t i) {
     return f32 ? reinterpret_cast<const float*>(pool)[i] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(pool)[i]);
 }
-// entry i of a vector whose first rot_dims entries are rotated in pairs (i, i + rot_dims / 2) by position `pos`
-__device__ __forceinline__ float rotate_half_at(const float* v, int i, int pos, const RotaryTable& rot) {
+// entry i of a vector whose first rot_dims entries are rotated by position `pos`, in pairs (i, i + rot_dims / 2) or (2i, 2i + 1)
+__device__ __forceinline__ float rotated_at(const float* v, int i, int pos, const RotaryTable& rot) {
     const int half = rot.rot_dims / 2;
     if (i >= rot.rot_dims) return v[i];
+    if (rot.pairs) {
+        const float cs = rot.cos[(size_t)pos * half + i / 2], sn = rot.sin[(size_t)pos * half + i / 2];
+        return i & 1 ? v[i] * cs + v[i - 1] * sn : v[i] * cs - v[i + 1] * sn;
+    }
     const int p = i < half ? i : i - half;
     const float cs = rot.cos[(size_t)pos * half + p], sn = rot.sin[(size_t)pos * half + p];
     return i < half ? v[i] * cs - v[i + half] * sn : v[i] * cs + v[i - half] * sn;
+}
+// entry i of a head's query in the coordinates of the cached rows
+__device__ __forceinline__ float query_at(const LatentAttnArgs& a, int t, int h, int i, int pos) {
+    if (a.q_raw && i >= a.rank) return rotated_at(a.q_raw + ((size_t)t * a.H + h) * (a.d + a.dr) + a.d, i - a.rank, pos, a.rot);
+    return a.qv[((size_t)t * a.H + h) * (a.rank + a.dr) + i];
 }
 }  // namespace
 
@@ -36,24 +46,34 @@ __device__ __forceinline__ float rotate_half_at(const float* v, int i, int pos, 
 __global__ void __launch_bounds__(128) latent_store_kernel(LatentAttnArgs a, RaggedDev r) {
     griddep_launch();
     griddep_wait();
-    __shared__ float red[4];
+    __shared__ float red[2][4];
     const int t = blockIdx.x, pos = r.tok_pos[t];
     const int slot = r.seg_slot[r.tok_seg[t]];
     const int Dk = a.rank + a.dr;
-    const float* dkv = a.proj + (size_t)t * a.ldp + a.dkv_off;
-    const size_t dst = ((size_t)a.block_tables[slot][pos / a.block_tokens] * a.block_tokens + pos % a.block_tokens) * Dk;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < a.rank; i += blockDim.x) ss = fmaf(dkv[i], dkv[i], ss);
-    ss = warp_sum(ss);
-    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    const bool own = a.dkv_off >= 0;
+    const float* dkv = a.proj + (size_t)t * a.ldp + (own ? a.dkv_off : 0);
+    const float* dq = a.proj + (size_t)t * a.ldp + a.dq_off;
+    float ss = 0.f, sq = 0.f;
+    if (own) for (int i = threadIdx.x; i < a.rank; i += blockDim.x) ss = fmaf(dkv[i], dkv[i], ss);
+    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) sq = fmaf(dq[i], dq[i], sq);
+    ss = warp_sum(ss); sq = warp_sum(sq);
+    if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = ss; red[1][threadIdx.x >> 5] = sq; }
     __syncthreads();
-    const float rinv = 1.f / sqrtf((red[0] + red[1] + red[2] + red[3]) / (float)a.rank + a.eps);
-    for (int i = threadIdx.x; i < a.rank; i += blockDim.x) row_store(a.pool, a.cache_f32, dst + i, dkv[i] * rinv * a.c_norm_w[i]);
-    for (int i = threadIdx.x; i < a.dr; i += blockDim.x) row_store(a.pool, a.cache_f32, dst + a.rank + i, rotate_half_at(dkv + a.rank, i, pos, a.rot));
+    if (own) {
+        const size_t dst = ((size_t)a.block_tables[slot][pos / a.block_tokens] * a.block_tokens + pos % a.block_tokens) * a.ld_row;
+        const float rinv = 1.f / sqrtf((red[0][0] + red[0][1] + red[0][2] + red[0][3]) / (float)a.rank + a.eps);
+        for (int i = threadIdx.x; i < a.rank; i += blockDim.x) row_store(a.pool, a.cache_f32, dst + i, dkv[i] * rinv * a.c_norm_w[i]);
+        for (int i = threadIdx.x; i < a.dr; i += blockDim.x) row_store(a.pool, a.cache_f32, dst + a.rank + i, rotated_at(dkv + a.rank, i, pos, a.rot));
+    }
+    if (a.q_rank > 0) {
+        const float rinv = 1.f / sqrtf((red[1][0] + red[1][1] + red[1][2] + red[1][3]) / (float)a.q_rank + a.eps);
+        for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) a.cq[(size_t)t * a.q_rank + i] = dq[i] * rinv * a.q_norm_w[i];
+        return;
+    }
     for (int j = threadIdx.x; j < a.H * a.dr; j += blockDim.x) {
         const int h = j / a.dr, i = j % a.dr;
         const float* q = a.proj + (size_t)t * a.ldp + a.q_off + (size_t)h * (a.d + a.dr) + a.d;
-        a.qv[((size_t)t * a.H + h) * Dk + a.rank + i] = rotate_half_at(q, i, pos, a.rot);
+        a.qv[((size_t)t * a.H + h) * Dk + a.rank + i] = rotated_at(q, i, pos, a.rot);
     }
 }
 cudaError_t latent_store_launch(const LatentAttnArgs& a, const RaggedDev& r, cudaStream_t s) {
@@ -61,7 +81,7 @@ cudaError_t latent_store_launch(const LatentAttnArgs& a, const RaggedDev& r, cud
 }
 
 // grid (T, H, splits), 8 warps: CTA z takes the z-th range of the visible keys, warp w its keys w, w + 8, ...; a lane holds
-// entries lane, lane + 32, ... of the row. The sink enters as the starting state of warp 0 of range 0: maximum = sink,
+// entries lane, lane + 32, ... of the row. A sink enters as the starting state of warp 0 of range 0: maximum = sink,
 // sum = 1, no value. With several ranges the CTA leaves (max, sum, unnormalised output) for latent_merge_kernel.
 constexpr int LA_WARPS = 8;
 template <int E>
@@ -74,19 +94,18 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(LatentAttnAr
     const int pos = r.tok_pos[t];
     const int* table = a.block_tables[r.seg_slot[r.tok_seg[t]]];
     const int Dk = a.rank + a.dr;
-    const float* q = a.qv + ((size_t)t * a.H + h) * Dk;
     float qr[E], acc[E];
 #pragma unroll
-    for (int e = 0; e < E; e++) { const int i = lane + 32 * e; qr[e] = i < Dk ? q[i] * a.scale : 0.f; acc[e] = 0.f; }
+    for (int e = 0; e < E; e++) { const int i = lane + 32 * e; qr[e] = i < Dk ? query_at(a, t, h, i, pos) * a.scale : 0.f; acc[e] = 0.f; }
     const int lo = max(0, pos - a.window + 1);
     const int n_splits = gridDim.z, n_all = pos - lo + 1, chunk = (n_all + n_splits - 1) / n_splits;
     const int j_begin = lo + blockIdx.z * chunk, j_end = min(pos + 1, j_begin + chunk);
-    const bool has_sink = warp == 0 && blockIdx.z == 0;
+    const bool has_sink = a.sink && warp == 0 && blockIdx.z == 0;
     float m = has_sink ? a.sink[h] : -INFINITY, l = has_sink ? 1.f : 0.f;
     for (int j0 = j_begin + warp * 2; j0 < j_end; j0 += LA_WARPS * 2) {       // two keys per round: their loads overlap
         const int j1 = min(j0 + 1, j_end - 1);
-        const size_t base0 = ((size_t)table[j0 / a.block_tokens] * a.block_tokens + j0 % a.block_tokens) * Dk;
-        const size_t base1 = ((size_t)table[j1 / a.block_tokens] * a.block_tokens + j1 % a.block_tokens) * Dk;
+        const size_t base0 = ((size_t)table[j0 / a.block_tokens] * a.block_tokens + j0 % a.block_tokens) * a.ld_row;
+        const size_t base1 = ((size_t)table[j1 / a.block_tokens] * a.block_tokens + j1 % a.block_tokens) * a.ld_row;
         float k0[E], k1[E], d0 = 0.f, d1 = 0.f;
 #pragma unroll
         for (int e = 0; e < E; e++) {
@@ -143,18 +162,17 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_pairs_kernel(Latent
     const int pos = r.tok_pos[t];
     const int* table = a.block_tables[r.seg_slot[r.tok_seg[t]]];
     const int Dk = a.rank + a.dr;
-    const float* q = a.qv + ((size_t)t * a.H + h) * Dk;
     float2 qr[E2], acc[E2];
 #pragma unroll
     for (int e = 0; e < E2; e++) {
         const int i = 64 * e + 2 * lane;
-        qr[e] = i < Dk ? make_float2(q[i] * a.scale, q[i + 1] * a.scale) : make_float2(0.f, 0.f);
+        qr[e] = i < Dk ? make_float2(query_at(a, t, h, i, pos) * a.scale, query_at(a, t, h, i + 1, pos) * a.scale) : make_float2(0.f, 0.f);
         acc[e] = make_float2(0.f, 0.f);
     }
     const int lo = max(0, pos - a.window + 1);
     const int n_splits = gridDim.z, n_all = pos - lo + 1, chunk = (n_all + n_splits - 1) / n_splits;
     const int j_begin = lo + blockIdx.z * chunk, j_end = min(pos + 1, j_begin + chunk);
-    const bool has_sink = warp == 0 && blockIdx.z == 0;
+    const bool has_sink = a.sink && warp == 0 && blockIdx.z == 0;
     float m = has_sink ? a.sink[h] : -INFINITY, l = has_sink ? 1.f : 0.f;
     for (int j0 = j_begin + warp * LA_KEYS; j0 < j_end; j0 += LA_WARPS * LA_KEYS) {
         size_t base[LA_KEYS];
@@ -163,7 +181,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_pairs_kernel(Latent
 #pragma unroll
         for (int u = 0; u < LA_KEYS; u++) {
             const int j = min(j0 + u, j_end - 1);          // past the end: the last key again, its weight is dropped below
-            base[u] = ((size_t)table[j / a.block_tokens] * a.block_tokens + j % a.block_tokens) * Dk;
+            base[u] = ((size_t)table[j / a.block_tokens] * a.block_tokens + j % a.block_tokens) * a.ld_row;
         }
 #pragma unroll
         for (int u = 0; u < LA_KEYS; u++)
@@ -222,7 +240,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_pairs_kernel(Latent
     }
 }
 
-// sum of the key ranges of one (token, head) in range order (range 0 carries the sink, so the sum is never empty)
+// sum of the key ranges of one (token, head) in range order (some range has keys, so the sum is never empty)
 __global__ void __launch_bounds__(128) latent_merge_kernel(LatentAttnArgs a, int n_splits) {
     griddep_launch();
     griddep_wait();
@@ -244,7 +262,7 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(LatentAttnArgs a, int
 // 256: every chunk recomputes the scores, so wide chunks pay back their registers); 4 warps x 16 query rows; cached rows in
 // blocks of 64, staged in shared memory once for all 64 queries. S = Q K^T over the whole row, O += P K[:, chunk], with
 // mma.sync m16n8k16 (bf16 in, f32 accumulate); mask, running maximum, exponentials and sums are 32-bit; the running state
-// starts at (maximum = sink, sum = 1).
+// starts at (maximum = sink, sum = 1) where there is a sink.
 constexpr int LT_Q = 64, LT_K = 64;
 namespace {
 __device__ __forceinline__ void cp_async_16z(void* smem_dst, const void* gsrc, int src_bytes) {
@@ -285,8 +303,7 @@ __global__ void __launch_bounds__(128) latent_attn_mma_kernel(LatentAttnArgs a, 
         const int rr = i / (Dk / 2), c = (i % (Dk / 2)) * 2;
         float2 v = make_float2(0.f, 0.f);
         if (rr < nq) {
-            const float* q = a.qv + ((size_t)(row0 + rr) * a.H + h) * Dk + c;
-            v = make_float2(q[0] * a.scale, q[1] * a.scale);
+            v = make_float2(query_at(a, row0 + rr, h, c, p0 + rr) * a.scale, query_at(a, row0 + rr, h, c + 1, p0 + rr) * a.scale);
         }
         *reinterpret_cast<__nv_bfloat162*>(Qs + rr * LD + c) = __floats2bfloat162_rn(v.x, v.y);
     }
@@ -294,7 +311,7 @@ __global__ void __launch_bounds__(128) latent_attn_mma_kernel(LatentAttnArgs a, 
     float o[LT_DV / 8][4];
 #pragma unroll
     for (int i = 0; i < LT_DV / 8; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-    const float sink = a.sink[h];
+    const float sink = a.sink ? a.sink[h] : -INFINITY;
     float m_run[2] = {sink, sink}, l_run[2] = {0.f, 0.f};      // the sink's own 1 joins the sum after the lane reduction
     const int gq = lane >> 2, tq = lane & 3;
     const int qrow[2] = {warp * 16 + gq, warp * 16 + gq + 8};
@@ -304,7 +321,7 @@ __global__ void __launch_bounds__(128) latent_attn_mma_kernel(LatentAttnArgs a, 
         for (int i = threadIdx.x; i < LT_K * (Dk / 8); i += blockDim.x) {
             const int rr = i / (Dk / 8), c = (i % (Dk / 8)) * 8;
             const int j = j0 + rr, jj = min(j, p_last);
-            const size_t base = ((size_t)table[jj / a.block_tokens] * a.block_tokens + jj % a.block_tokens) * Dk + c;
+            const size_t base = ((size_t)table[jj / a.block_tokens] * a.block_tokens + jj % a.block_tokens) * a.ld_row + c;
             cp_async_16z(Ks + rr * LD + c, pool + base, j <= p_last ? 16 : 0);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -336,13 +353,14 @@ __global__ void __launch_bounds__(128) latent_attn_mma_kernel(LatentAttnArgs a, 
                 sacc[ni][e] = v;
                 mx[e >> 1] = fmaxf(mx[e >> 1], v);
             }
-        float corr[2];
+        float corr[2], m_ref[2];
 #pragma unroll
         for (int q2 = 0; q2 < 2; q2++) {
             mx[q2] = fmaxf(mx[q2], __shfl_xor_sync(0xffffffffu, mx[q2], 1));
             mx[q2] = fmaxf(mx[q2], __shfl_xor_sync(0xffffffffu, mx[q2], 2));
-            const float m_new = fmaxf(m_run[q2], mx[q2]);       // finite: the sink is
-            corr[q2] = expf(m_run[q2] - m_new);
+            const float m_new = fmaxf(m_run[q2], mx[q2]);
+            m_ref[q2] = m_new > -INFINITY ? m_new : 0.f;        // a row that has seen no key yet (no sink): all weights stay 0
+            corr[q2] = expf(m_run[q2] - m_ref[q2]);
             m_run[q2] = m_new;
             l_run[q2] *= corr[q2];
         }
@@ -350,7 +368,7 @@ __global__ void __launch_bounds__(128) latent_attn_mma_kernel(LatentAttnArgs a, 
         for (int ni = 0; ni < LT_K / 8; ni++)
 #pragma unroll
             for (int e = 0; e < 4; e++) {
-                const float pv = expf(sacc[ni][e] - m_run[e >> 1]);
+                const float pv = expf(sacc[ni][e] - m_ref[e >> 1]);
                 sacc[ni][e] = pv;
                 l_run[e >> 1] += pv;
             }
@@ -378,7 +396,7 @@ __global__ void __launch_bounds__(128) latent_attn_mma_kernel(LatentAttnArgs a, 
     for (int q2 = 0; q2 < 2; q2++) {
         l_run[q2] += __shfl_xor_sync(0xffffffffu, l_run[q2], 1);
         l_run[q2] += __shfl_xor_sync(0xffffffffu, l_run[q2], 2);
-        l_run[q2] += expf(sink - m_run[q2]);
+        if (a.sink) l_run[q2] += expf(sink - m_run[q2]);
     }
 #pragma unroll
     for (int i = 0; i < LT_DV / 8; i++)
@@ -393,7 +411,7 @@ cudaError_t latent_attn_launch(const LatentAttnArgs& a, const RaggedDev& r, cuda
     const int Dk = a.rank + a.dr;
     if (Dk > 640) return cudaErrorInvalidValue;
     static const bool no_mma = getenv("B2_NO_ATTN_MMA") != nullptr;        // tuning aid: scalar attention for prompts too
-    if (!no_mma && !a.cache_f32 && r.T > 8 && a.rank % 16 == 0 && Dk % 16 == 0) {
+    if (!no_mma && !a.cache_f32 && r.T > 8 && a.rank % 16 == 0 && Dk % 16 == 0 && a.ld_row % 8 == 0) {
         static bool attr_done = false;
         if (!attr_done) {
             cudaFuncSetAttribute(latent_attn_mma_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * 64 * (640 + 8) * 2);
@@ -413,7 +431,7 @@ cudaError_t latent_attn_launch(const LatentAttnArgs& a, const RaggedDev& r, cuda
     const dim3 grid(r.T, a.H, splits), block(LA_WARPS * 32);
     const size_t smem = (size_t)LA_WARPS * a.rank * 4;
     cudaError_t ce;
-    if (Dk % 2 == 0) {
+    if (Dk % 2 == 0 && a.ld_row % 2 == 0) {
         if (Dk <= 192) ce = a.cache_f32 ? launch_chain(latent_attn_pairs_kernel<3, true>, grid, block, smem, s, a, r)
                                         : launch_chain(latent_attn_pairs_kernel<3, false>, grid, block, smem, s, a, r);
         else if (Dk <= 384) ce = a.cache_f32 ? launch_chain(latent_attn_pairs_kernel<6, true>, grid, block, smem, s, a, r)

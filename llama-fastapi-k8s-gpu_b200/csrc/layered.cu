@@ -2,11 +2,12 @@
 // layers over dense bf16 / f32 tensors, stepped over ragged batches. Token mixers: window attention beside a selective
 // scan, an mLSTM matrix memory, latent attention, the gated delta rule, a Mamba-2 state-space layer, chunk-local sigmoid
 // attention beside fixed-decay linear attention, softmax attention with a sink alone or beside a head-decay delta rule.
-// Feed-forward blocks: squared ReLU with biases, a gated SiLU unit, a block with a piecewise activation, or a routed mixture of
-// gated experts (SiLU or clamped; with an optional shared expert). Four block styles: layer norm AFTER each residual sum,
-// pre-norm (zero-centred RMS weights) with a scaled branch, an RMS norm in parts on each branch's OUTPUT, or pre-norm over
-// several copies of the stream with mixing matrices and a convolution on every sublayer's input. A layer entry may name another
-// layer's tensors (a repeated run of layers: shared weights, cache and state of its own). Shares the engine object with the
+// Feed-forward blocks: squared ReLU with biases, a gated SiLU or GELU unit, a block with a piecewise activation, or a routed
+// mixture of gated experts (SiLU or clamped; with an optional shared expert). Five block styles: layer norm AFTER each residual
+// sum, pre-norm (zero-centred RMS weights) with a scaled branch, an RMS norm in parts on each branch's OUTPUT, pre-norm over
+// several copies of the stream with mixing matrices and a convolution on every sublayer's input, or parallel sublayers behind two
+// layer norms of the same stream. A layer entry may name another layer's tensors (a repeated run of layers: shared weights, cache
+// and state of its own); a latent-attention layer may read the rows another layer caches. Shares the engine object with the
 // llama graph (engine.cu): tensors, sequence slots and their page tables, sampler state, stream, error reporting. Owns: fused
 // projection matrices, per-layer cache pages, per-slot recurrent state, the step workspace.
 #include "engine_state.h"
@@ -25,7 +26,7 @@ struct DenseW { const void* w = nullptr; int type = 0, N = 0, K = 0; };
 
 struct LyLayer {
     b2_layer_desc d = {};
-    float *norm1 = nullptr, *norm2 = nullptr;
+    float *norm1 = nullptr, *norm2 = nullptr, *norm1_b = nullptr, *norm2_b = nullptr;
     // window attention + selective scan
     DenseW in_proj, attn_o, scan_x, scan_dt, scan_o;      // in_proj rows: q | k | x | z
     int q_off = 0, k_off = 0, x_off = 0, z_off = 0;
@@ -42,10 +43,11 @@ struct LyLayer {
     // feed-forward
     DenseW up, down;
     float *up_b = nullptr, *down_b = nullptr;
-    // latent attention: la_proj rows q | dkv | g; uk_t = W_uk transposed per head [H][rank][d]
-    DenseW la_proj, uk_t, uv;
-    int g_off = 0, dkv_off = 0;
-    float *c_norm = nullptr, *sink = nullptr;
+    // latent attention: la_proj rows q (or dq) | dkv | g, absent ones left out; uk_t = W_uk transposed per head [H][rank][d]; uq: from
+    // the query latent to the queries
+    DenseW la_proj, uk_t, uv, uq;
+    int g_off = 0, dkv_off = 0, la_row = 0;    // la_row: entries of a cached row (of the layer that owns the pages)
+    float *c_norm = nullptr, *sink = nullptr, *dq_norm = nullptr;
     void* la_pool = nullptr;
     // delta rule (st_proj rows q | k | v | b | a1 | g1) and state-space layer (st_proj rows z | x | B | C | dt)
     DenseW st_proj, a2, g2, ag, st_o;                      // ag: a2 and g2 as one block-diagonal matrix over the input a1 | g1
@@ -79,18 +81,18 @@ struct LayeredModel {
     b2_layered_config c = {};
     std::vector<LyLayer> layers;
     std::vector<void*> owned;          // device allocations freed at destroy
-    DenseW embed, head;
-    float *final_norm = nullptr, *embed_norm = nullptr;
+    DenseW embed, head, bigram;
+    float *final_norm = nullptr, *final_norm_b = nullptr, *embed_norm = nullptr;
     bool exact = false;                // B2_FLAG_F32
     int** block_tables = nullptr;      // device [max_seqs] -> page table
     // step workspace (max_step_tokens rows)
     float *xs = nullptr, *hc = nullptr, *cross = nullptr;     // copies of the stream [S][max_step_tokens][W]; convolved sublayer input; per-(query head, value head) attention sums
-    float *x = nullptr, *proj = nullptr, *buf[4] = {}, *oL = nullptr, *oR = nullptr, *hn = nullptr, *ff = nullptr, *rows = nullptr, *logits = nullptr;
+    float *x = nullptr, *proj = nullptr, *buf[4] = {}, *oL = nullptr, *oR = nullptr, *hn = nullptr, *hn2 = nullptr, *ff = nullptr, *rows = nullptr, *logits = nullptr;
     __nv_bfloat16* xb = nullptr;       // a product's input rounded to bf16 [max_step_tokens][widest input]
     std::unordered_map<std::string, StepGraph> graphs;     // replayable small steps, by shape (b2_step)
     bool graphs_on = true;
     // mixture of experts: router outputs, choices, the sorted pair table, expert activations and outputs
-    float *moe_logits = nullptr, *moe_weight = nullptr, *moe_h = nullptr, *moe_y = nullptr;
+    float *moe_logits = nullptr, *moe_weight = nullptr, *moe_row_weight = nullptr, *moe_h = nullptr, *moe_y = nullptr;
     int *moe_sel = nullptr, *moe_tok = nullptr, *moe_pos = nullptr, *moe_rows = nullptr, *moe_tiles = nullptr;
     int moe_max_tiles = 0;
     float* attn_pbuf = nullptr;        // prompts with mixed heads: normalised attention weights of a group of query tiles
@@ -275,6 +277,9 @@ int layered_finalize(b2_engine* e) {
     if (c.tie_head) m->head = m->embed;
     else if ((rc = matrix(e, "head", V, W, m->head))) return rc;
     if ((rc = vec_f32(e, m, "final.norm", W, 1, &m->final_norm))) return rc;
+    const bool parallel = c.block_style == B2_BLOCK_PARALLEL_LN;
+    if (parallel && (rc = vec_f32(e, m, "final.norm.b", W, 1, &m->final_norm_b))) return rc;
+    if (c.bigram_buckets > 0 && (rc = matrix(e, "bigram", c.bigram_buckets + 1, W, m->bigram))) return rc;
     if (c.block_style == B2_BLOCK_PRENORM_RMS && (rc = vec_f32(e, m, "embed.norm", W, 1, &m->embed_norm))) return rc;
     const size_t cache_esz = m->exact ? 4 : 2;
     size_t max_proj = 1, max_buf = 1, max_ff = 1, max_attn = 0, max_attn_d = 0, max_glu = 0;
@@ -325,6 +330,10 @@ int layered_finalize(b2_engine* e) {
             }
         }
         if ((rc = vec_f32(e, m, p + "norm1", W, 1, &L.norm1))) return rc;
+        if (parallel) {
+            if ((rc = vec_f32(e, m, p + "norm1.b", W, 1, &L.norm1_b))) return rc;
+            if (d.n_ff > 0 && (rc = vec_f32(e, m, p + "norm2.b", W, 1, &L.norm2_b))) return rc;
+        }
         if (hyper) {
             for (int q = 0; q < (d.n_ff > 0 ? 2 : 1); q++) {
                 const std::string hc = p + "hc" + std::to_string(q + 1) + ".";
@@ -413,11 +422,19 @@ int layered_finalize(b2_engine* e) {
         } else if (d.mixer == B2_MIX_LATENT_ATTN) {
             const std::string a = p + "mix.";
             const int H = d.n_head, dq = d.head_dim + d.la_rot_dim, Dk = d.la_rank + d.la_rot_dim, vd = H * d.la_vdim;
+            const bool own = d.kv_from == 0, gate = !(d.attn_flags & B2_ATTN_NO_GATE);
+            std::vector<std::pair<std::string, int>> parts = {d.la_q_rank > 0 ? std::make_pair(a + "dq", d.la_q_rank) : std::make_pair(a + "q", H * dq)};
+            if (own) parts.push_back({a + "dkv", Dk});
+            if (gate) parts.push_back({a + "g", (d.attn_flags & B2_ATTN_HEAD_GATE) ? H : vd});
             std::vector<int> offs;
-            if ((rc = fuse(e, m, {{a + "q", H * dq}, {a + "dkv", Dk}, {a + "g", vd}}, W, L.la_proj, offs))) return rc;
-            L.q_off = offs[0]; L.dkv_off = offs[1]; L.g_off = offs[2];
-            if ((rc = vec_f32(e, m, a + "dkv.norm", d.la_rank, 1, &L.c_norm))) return rc;
-            if ((rc = vec_f32(e, m, a + "sink", H, 1, &L.sink))) return rc;
+            if ((rc = fuse(e, m, parts, W, L.la_proj, offs))) return rc;
+            L.q_off = offs[0]; L.dkv_off = own ? offs[1] : -1; L.g_off = gate ? offs.back() : 0;
+            if (d.la_q_rank > 0) {
+                if ((rc = vec_f32(e, m, a + "dq.norm", d.la_q_rank, 1, &L.dq_norm))) return rc;
+                if ((rc = matrix(e, a + "uq", H * dq, d.la_q_rank, L.uq))) return rc;
+            }
+            if (own && (rc = vec_f32(e, m, a + "dkv.norm", d.la_rank, 1, &L.c_norm))) return rc;
+            if (!(d.attn_flags & B2_ATTN_NO_SINK) && (rc = vec_f32(e, m, a + "sink", H, 1, &L.sink))) return rc;
             DenseW uk;
             if ((rc = matrix(e, a + "uk", H * d.head_dim, d.la_rank, uk))) return rc;
             {
@@ -433,11 +450,17 @@ int layered_finalize(b2_engine* e) {
             L.uv.N = d.la_vdim;                       // applied head by head
             if ((rc = matrix(e, a + "o", W, vd, L.attn_o))) return rc;
             if ((rc = build_rotary(e, m, L))) return rc;
-            const size_t pool = (size_t)c.kv_num_blocks * c.kv_block_tokens * Dk * cache_esz;
-            if ((rc = dev_alloc(m, &L.la_pool, pool, true))) return rc;
-            e->kv_bytes += (int64_t)pool;
+            if (own) {
+                const size_t pool = (size_t)c.kv_num_blocks * c.kv_block_tokens * Dk * cache_esz;
+                if ((rc = dev_alloc(m, &L.la_pool, pool, true))) return rc;
+                e->kv_bytes += (int64_t)pool;
+                L.la_row = Dk;
+            } else {
+                L.la_pool = m->layers[d.kv_from - 1].la_pool;
+                L.la_row = m->layers[d.kv_from - 1].la_row;
+            }
             max_proj = std::max<size_t>(max_proj, L.la_proj.N);
-            max_buf = std::max<size_t>({max_buf, (size_t)H * Dk, (size_t)H * dq, (size_t)vd});
+            max_buf = std::max<size_t>({max_buf, (size_t)H * Dk, (size_t)H * dq, (size_t)vd, (size_t)d.la_q_rank});
             max_attn = 1; max_attn_d = std::max<size_t>(max_attn_d, d.la_rank);
         } else if (d.mixer == B2_MIX_CHUNK_LINEAR) {
             const std::string a = p + "mix.left.", b = p + "mix.right.";
@@ -535,7 +558,7 @@ int layered_finalize(b2_engine* e) {
             if ((rc = vec_f32(e, m, p + "norm2", W, 1, &L.norm2))) return rc;
             if ((rc = matrix(e, p + "mlp.router", slots, W, L.router))) return rc;
             const std::string cn = p + (d.moe_route == B2_ROUTE_TOPK_SOFTMAX ? "mlp.router.b" : "mlp.correction");
-            if ((!hyper || e->tensors.count(cn)) && (rc = vec_f32(e, m, cn, slots, 1, &L.correction))) return rc;
+            if ((!(hyper || d.moe_route == B2_ROUTE_SIGMOID) || e->tensors.count(cn)) && (rc = vec_f32(e, m, cn, slots, 1, &L.correction))) return rc;
             if ((rc = stack_experts(e, m, p + "mlp.e", d.moe_experts, d.n_ff, W, L.gate_up, L.e_down))) return rc;
             if (d.moe_shared_ff > 0) {
                 if ((rc = stack_experts(e, m, p + "mlp.shared", 0, d.moe_shared_ff, W, L.glu_gate_up, L.glu_down))) return rc;
@@ -586,6 +609,7 @@ int layered_finalize(b2_engine* e) {
     if ((rc = dev_alloc(m, (void**)&m->oL, (size_t)Tm * W * 4))) return rc;
     if ((rc = dev_alloc(m, (void**)&m->oR, (size_t)Tm * W * 4))) return rc;
     if ((rc = dev_alloc(m, (void**)&m->hn, (size_t)Tm * W * 4))) return rc;
+    if (parallel && (rc = dev_alloc(m, (void**)&m->hn2, (size_t)Tm * W * 4))) return rc;
     max_ff = std::max(max_ff, max_glu);
     if ((rc = dev_alloc(m, (void**)&m->ff, (size_t)Tm * max_ff * 4))) return rc;
     if (!m->exact && (rc = dev_alloc(m, (void**)&m->xb, (size_t)(Tm + B2_STEP_MAX_ENTRIES) * std::max<size_t>({max_buf, max_ff, (size_t)W, moe_xb}) * 2 + 64))) return rc;
@@ -600,6 +624,7 @@ int layered_finalize(b2_engine* e) {
         m->moe_max_tiles = (int)(moe_pairs / 64 + moe_experts + 1);
         if ((rc = dev_alloc(m, (void**)&m->moe_logits, (size_t)Tm * moe_slots * 4))) return rc;
         if ((rc = dev_alloc(m, (void**)&m->moe_weight, moe_pairs * 4))) return rc;
+        if ((rc = dev_alloc(m, (void**)&m->moe_row_weight, moe_pairs * 4))) return rc;
         if ((rc = dev_alloc(m, (void**)&m->moe_sel, moe_pairs * 4))) return rc;
         if ((rc = dev_alloc(m, (void**)&m->moe_tok, moe_pairs * 4))) return rc;
         if ((rc = dev_alloc(m, (void**)&m->moe_pos, moe_pairs * 4))) return rc;
@@ -610,7 +635,7 @@ int layered_finalize(b2_engine* e) {
     }
     if ((rc = dev_alloc(m, (void**)&m->rows, (size_t)LOGIT_ROWS * W * 4))) return rc;
     if ((rc = dev_alloc(m, (void**)&m->logits, (size_t)LOGIT_ROWS * V * 4))) return rc;
-    const size_t n_meta = (size_t)4 * Tm + 2 * (Tm / 64 + B2_STEP_MAX_ENTRIES) + 5 * B2_STEP_MAX_ENTRIES + 64;
+    const size_t n_meta = (size_t)5 * Tm + 2 * (Tm / 64 + B2_STEP_MAX_ENTRIES) + 5 * B2_STEP_MAX_ENTRIES + 64;
     if ((rc = dev_alloc(m, (void**)&m->meta, n_meta * 4))) return rc;
     CK(cudaMallocHost(&m->meta_host, n_meta * 4));
     CK(cudaMallocHost(&m->logits_host, (size_t)LOGIT_ROWS * V * 4));
@@ -704,6 +729,14 @@ extern "C" int b2_engine_create_layered(const b2_layered_config* c, const b2_lay
             if (d.n_head <= 0 || d.head_dim <= 0 || d.la_rot_dim < 0 || d.la_vdim <= 0 || d.la_rank <= 0) return b2_fail(B2_ERR_ARG, li + "bad latent-attention sizes");
             if (d.rot_dims < 0 || d.rot_dims > d.la_rot_dim || d.rot_dims % 2) return b2_fail(B2_ERR_ARG, li + "rotary dims must be even and <= the rotated part");
             if (d.la_rank + d.la_rot_dim > 640) return b2_fail(B2_ERR_UNSUPPORTED, li + "latent + rotated key part above 640");
+            if (d.la_q_rank < 0) return b2_fail(B2_ERR_ARG, li + "negative query latent");
+            if (d.kv_from < 0 || d.kv_from > i) return b2_fail(B2_ERR_ARG, li + "kv_from must name an earlier layer");
+            if (d.kv_from > 0) {
+                const b2_layer_desc& o = layers[d.kv_from - 1];
+                if (o.mixer != B2_MIX_LATENT_ATTN || o.kv_from > 0 || o.la_rank != d.la_rank || d.la_rot_dim > 0)
+                    return b2_fail(B2_ERR_ARG, li + "kv_from must name a latent-attention layer with rows of its own and the same latent size, and takes no rotated part");
+                if (d.la_q_rank == 0) return b2_fail(B2_ERR_UNSUPPORTED, li + "kv_from needs queries through a latent");
+            }
         } else if (d.mixer == B2_MIX_DELTA_RULE) {
             if (d.mm_heads <= 0 || d.key_heads <= 0 || d.mm_heads % d.key_heads || d.mm_dim <= 0 || d.mm_vdim <= 0 || d.rank_a <= 0 || d.rank_g <= 0 ||
                 d.conv_taps <= 0 || d.conv_taps > 64)
@@ -737,17 +770,18 @@ extern "C" int b2_engine_create_layered(const b2_layered_config* c, const b2_lay
                 d.moe_keep <= 0 || d.moe_keep > d.moe_groups || d.moe_top > d.moe_keep * (slots / d.moe_groups))
                 return b2_fail(B2_ERR_ARG, li + "bad mixture-of-experts sizes");
             if (slots > 4096) return b2_fail(B2_ERR_UNSUPPORTED, li + "more than 4096 expert slots");
-            if (d.moe_route != B2_ROUTE_SOFTMAX_ALL && d.moe_route != B2_ROUTE_TOPK_SOFTMAX) return b2_fail(B2_ERR_ARG, li + "unknown routing rule");
+            if (d.moe_route != B2_ROUTE_SOFTMAX_ALL && d.moe_route != B2_ROUTE_TOPK_SOFTMAX && d.moe_route != B2_ROUTE_SIGMOID) return b2_fail(B2_ERR_ARG, li + "unknown routing rule");
             if (d.moe_route == B2_ROUTE_TOPK_SOFTMAX && (d.moe_identity > 0 || d.moe_groups > 1)) return b2_fail(B2_ERR_UNSUPPORTED, li + "top-k softmax routing has no identity slots or groups");
+            if (d.moe_scale_input && d.moe_identity > 0) return b2_fail(B2_ERR_UNSUPPORTED, li + "identity slots have no scaled input");
             if (d.moe_shared_ff < 0) return b2_fail(B2_ERR_ARG, li + "negative shared-expert width");
             if (d.moe_expert != B2_EXPERT_SILU && d.moe_expert != B2_EXPERT_CLAMPED) return b2_fail(B2_ERR_ARG, li + "unknown expert kind");
             if (d.moe_expert == B2_EXPERT_CLAMPED && !(d.moe_limit > 0.0)) return b2_fail(B2_ERR_ARG, li + "a clamped expert needs a positive limit");
         } else if (d.ff_kind != B2_FF_RELU2 && d.ff_kind != B2_FF_GLU && d.ff_kind != B2_FF_PIECEWISE) return b2_fail(B2_ERR_UNSUPPORTED, li + "unknown feed-forward kind");
-        if (c->block_style == B2_BLOCK_PRENORM_RMS ? (d.mixer == B2_MIX_WINDOW_SCAN) : false)
+        if (d.ff_act != B2_ACT_SILU && d.ff_act != B2_ACT_GELU_TANH) return b2_fail(B2_ERR_ARG, li + "unknown activation");
+        if ((c->block_style == B2_BLOCK_PRENORM_RMS || c->block_style == B2_BLOCK_PARALLEL_LN) && d.mixer == B2_MIX_WINDOW_SCAN)
             return b2_fail(B2_ERR_UNSUPPORTED, li + "the two-branch mixer belongs to post-sum blocks");
     }
-    if (c->block_style != B2_BLOCK_POSTSUM_LN && c->block_style != B2_BLOCK_PRENORM_RMS && c->block_style != B2_BLOCK_OUTNORM_RMS &&
-        c->block_style != B2_BLOCK_HYPER_RMS)
+    if (c->block_style < B2_BLOCK_POSTSUM_LN || c->block_style > B2_BLOCK_PARALLEL_LN)
         return b2_fail(B2_ERR_ARG, "unknown block style");
     if (c->block_style == B2_BLOCK_HYPER_RMS) {
         if (c->n_streams < 0 || c->n_streams > 16) return b2_fail(B2_ERR_UNSUPPORTED, "at most 16 copies of the stream");
@@ -758,6 +792,7 @@ extern "C" int b2_engine_create_layered(const b2_layered_config* c, const b2_lay
     }
     if (c->block_style == B2_BLOCK_OUTNORM_RMS && (c->norm_groups < 0 || (c->norm_groups > 0 && c->n_embd % c->norm_groups)))
         return b2_fail(B2_ERR_ARG, "the norm's parts must divide the width");
+    if (c->bigram_buckets < 0 || c->bigram_mul_prev < 0 || c->bigram_mul_cur < 0) return b2_fail(B2_ERR_ARG, "bad bigram embedding");
     b2_engine* e = new b2_engine();
     b2_config& b = e->cfg;
     memset(&b, 0, sizeof(b));
@@ -901,8 +936,9 @@ static int mix_latent_attn(b2_engine* e, LayeredModel* m, LyLayer& L, const Ragg
     if ((rc = dense(e, m, L.la_proj, in, W, m->proj, Np, T))) return rc;
     LatentAttnArgs a = {};
     a.proj = m->proj; a.ldp = Np; a.q_off = L.q_off; a.dkv_off = L.dkv_off; a.c_norm_w = L.c_norm;
-    a.rot.cos = L.rot_cos; a.rot.sin = L.rot_sin; a.rot.rot_dims = d.rot_dims;
-    a.pool = L.la_pool; a.cache_f32 = m->exact ? 1 : 0; a.block_tables = m->block_tables; a.block_tokens = c.kv_block_tokens;
+    a.rot.cos = L.rot_cos; a.rot.sin = L.rot_sin; a.rot.rot_dims = d.rot_dims; a.rot.pairs = (d.attn_flags & B2_ATTN_ROT_PAIRS) ? 1 : 0;
+    a.dq_off = L.q_off; a.q_rank = d.la_q_rank; a.q_norm_w = L.dq_norm; a.cq = m->buf[3];
+    a.pool = L.la_pool; a.ld_row = L.la_row; a.cache_f32 = m->exact ? 1 : 0; a.block_tables = m->block_tables; a.block_tokens = c.kv_block_tokens;
     a.H = H; a.d = d.head_dim; a.dr = d.la_rot_dim; a.rank = d.la_rank; a.window = d.window > 0 ? d.window : c.n_ctx;
     a.scale = (float)d.attn_scale; a.eps = c.norm_eps; a.sink = L.sink; a.qv = m->buf[0]; a.o_lat = m->buf[1];
     a.split_scratch = m->attn_split; a.split_capacity = m->attn_split_floats;
@@ -911,20 +947,28 @@ static int mix_latent_attn(b2_engine* e, LayeredModel* m, LyLayer& L, const Ragg
         CK(latent_store_launch(a, r, st));
         e->launches++;
     }
+    const float* q = m->proj + L.q_off;
+    int ldq = Np;
+    if (d.la_q_rank > 0) {                  // the normed query latent, expanded; the attention rotates what it reads of it
+        if ((rc = dense(e, m, L.uq, m->buf[3], d.la_q_rank, m->buf[2], H * dq, T))) return rc;
+        a.q_raw = q = m->buf[2];
+        ldq = H * dq;
+    }
     // every head's unrotated query through its transposed key map: the head's query in the latent's coordinates
     DenseArgs b = {};
     b.batch = H; b.x_bs = dq; b.w_bs = (long)d.la_rank * d.head_dim; b.y_bs = Dk; b.x_span = H * dq;
-    if ((rc = dense(e, m, L.uk_t, m->proj + L.q_off, Np, m->buf[0], H * Dk, T, nullptr, EPI_NONE, 1, &b))) return rc;
+    if ((rc = dense(e, m, L.uk_t, q, ldq, m->buf[0], H * Dk, T, nullptr, EPI_NONE, 1, &b))) return rc;
     {
         StepProfiler sp(m, st, 2);
         CK(latent_attn_launch(a, r, st));
         e->launches += 2;
     }
-    // values of the weighted latent sums, head by head, times the sigmoid output gate
+    // values of the weighted latent sums, head by head, times the sigmoid output gate (one number per entry or per head)
+    const bool gate = !(d.attn_flags & B2_ATTN_NO_GATE), head_gate = (d.attn_flags & B2_ATTN_HEAD_GATE) != 0;
     DenseArgs v = {};
     v.batch = H; v.x_bs = d.la_rank; v.w_bs = (long)d.la_vdim * d.la_rank; v.y_bs = d.la_vdim; v.x_span = H * d.la_rank;
-    v.aux = m->proj + L.g_off; v.ldaux = Np; v.aux_bs = d.la_vdim;
-    if ((rc = dense(e, m, L.uv, m->buf[1], H * d.la_rank, m->buf[2], H * d.la_vdim, T, nullptr, EPI_MUL_SIGMOID, 1, &v))) return rc;
+    if (gate) { v.aux = m->proj + L.g_off; v.ldaux = Np; v.aux_bs = head_gate ? 1 : d.la_vdim; v.aux_one = head_gate; }
+    if ((rc = dense(e, m, L.uv, m->buf[1], H * d.la_rank, m->buf[2], H * d.la_vdim, T, nullptr, gate ? EPI_MUL_SIGMOID : EPI_NONE, 1, &v))) return rc;
     return dense(e, m, L.attn_o, m->buf[2], H * d.la_vdim, m->oL, W, T);
 }
 
@@ -1104,32 +1148,34 @@ static int mix_sink(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& 
     return dense(e, m, L.st_o, m->buf[2], vd, m->oR, W, T);
 }
 
-// ---- feed-forward blocks: input `in` [T][W], output in m->oL
-static int ff_piecewise(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in) {
+// ---- feed-forward blocks: input `in` [T][W], output `out` [T][W]
+static int ff_piecewise(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in, float* out) {
     const int T = r.T, W = m->c.n_embd;
     DenseArgs up = {};
     up.p0 = L.act_p0; up.p1 = L.act_p1;
     int rc;
     if ((rc = dense(e, m, L.up, in, W, m->ff, L.d.n_ff, T, nullptr, EPI_PIECEWISE, 1, &up))) return rc;
-    return dense(e, m, L.down, m->ff, L.d.n_ff, m->oL, W, T);
+    return dense(e, m, L.down, m->ff, L.d.n_ff, out, W, T);
 }
 
-static int ff_relu2(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in) {
+static int ff_relu2(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in, float* out) {
     const int T = r.T, W = m->c.n_embd;
     int rc;
     if ((rc = dense(e, m, L.up, in, W, m->ff, L.d.n_ff, T, L.up_b, EPI_BIAS_RELU2))) return rc;
-    return dense(e, m, L.down, m->ff, L.d.n_ff, m->oL, W, T, L.down_b, EPI_BIAS);
+    return dense(e, m, L.down, m->ff, L.d.n_ff, out, W, T, L.down_b, EPI_BIAS);
 }
 
-static int ff_glu(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in) {
+static int ff_glu(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in, float* out) {
     const int T = r.T, W = m->c.n_embd, ff = L.glu_down.K;
     int rc;
-    if ((rc = dense(e, m, L.glu_gate_up, in, W, m->ff, ff, T, nullptr, EPI_GLU_SILU))) return rc;
-    return dense(e, m, L.glu_down, m->ff, ff, m->oL, W, T);
+    // ff_act belongs to the dense block; a mixture's shared expert is a SiLU unit
+    const int epi = L.d.ff_kind == B2_FF_GLU && L.d.ff_act == B2_ACT_GELU_TANH ? EPI_GLU_GELU : EPI_GLU_SILU;
+    if ((rc = dense(e, m, L.glu_gate_up, in, W, m->ff, ff, T, nullptr, epi))) return rc;
+    return dense(e, m, L.glu_down, m->ff, ff, out, W, T);
 }
 
 // defer != nullptr: the weighted sum of the expert outputs is left to the caller's residual kernel (described in *defer)
-static int ff_moe(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in, MoeJoinArgs* defer) {
+static int ff_moe(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in, float* out, MoeJoinArgs* defer) {
     const b2_layer_desc& d = L.d;
     cudaStream_t st = e->stream;
     const int T = r.T, W = m->c.n_embd, slots = d.moe_experts + d.moe_identity, pairs = T * d.moe_top, ff = d.n_ff;
@@ -1140,7 +1186,7 @@ static int ff_moe(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r,
     MoeRouteArgs ra = {};
     ra.logits = m->moe_logits; ra.ld = slots; ra.correction = L.correction; ra.n_slots = slots; ra.n_experts = d.moe_experts;
     ra.top = d.moe_top; ra.n_groups = d.moe_groups; ra.keep_groups = d.moe_keep; ra.scale = (float)d.moe_scale;
-    ra.mode = d.moe_route == B2_ROUTE_TOPK_SOFTMAX ? 1 : 0; ra.renorm = d.moe_renorm;
+    ra.mode = d.moe_route == B2_ROUTE_TOPK_SOFTMAX ? 1 : d.moe_route == B2_ROUTE_SIGMOID ? 2 : 0; ra.renorm = d.moe_renorm;
     ra.sel = m->moe_sel; ra.weight = m->moe_weight; ra.pair_token = m->moe_tok;
     DenseGroups g = {};
     g.n_groups = d.moe_experts;
@@ -1157,29 +1203,33 @@ static int ff_moe(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r,
             sa.sel = m->moe_sel; sa.n_pairs = pairs; sa.top = d.moe_top; sa.n_experts = d.moe_experts; sa.tile = g.tile_max; sa.pos = m->moe_pos; sa.x_rows = m->moe_rows;
             sa.n_tiles = m->moe_tiles; sa.tile_group = m->moe_tiles + 1; sa.tile_row0 = sa.tile_group + m->moe_max_tiles;
             sa.tile_rows = sa.tile_row0 + m->moe_max_tiles; sa.max_tiles = m->moe_max_tiles;
+            if (d.moe_scale_input) { sa.weight = m->moe_weight; sa.row_weight = m->moe_row_weight; }
             CK(moe_sort_launch(sa, st));
             e->launches++;
             g.tile_group = sa.tile_group; g.tile_row0 = sa.tile_row0; g.tile_rows = sa.tile_rows; g.n_tiles = sa.n_tiles;
             g.max_tiles = std::min(m->moe_max_tiles, pairs / g.tile_max + d.moe_experts + 1);
         } else g.group = m->moe_sel;
     }
+    // weights on the inputs: w (W h) for W (w h), inside the epilogue before the activation; the outputs then add up as they are
+    const float* out_weight = d.moe_scale_input ? nullptr : m->moe_weight;
+    if (d.moe_scale_input) g.row_scale = tiled ? m->moe_row_weight : m->moe_weight;
     DenseArgs up = {};
     g.x_rows = tiled ? m->moe_rows : m->moe_tok; g.w_stride = (long)2 * ff * W; g.x_total_rows = T;
     up.groups = &g;
     up.p0 = (float)d.moe_limit; up.p1 = (float)d.moe_alpha;
     if ((rc = dense(e, m, L.gate_up, in, W, m->moe_h, ff, pairs, nullptr, d.moe_expert == B2_EXPERT_CLAMPED ? EPI_GLU_CLAMP : EPI_GLU_SILU, 1, &up))) return rc;
     DenseGroups g2 = g;
-    g2.x_rows = nullptr; g2.w_stride = (long)W * ff; g2.x_total_rows = pairs;
+    g2.x_rows = nullptr; g2.row_scale = nullptr; g2.w_stride = (long)W * ff; g2.x_total_rows = pairs;
     DenseArgs dn = {};
     dn.groups = &g2;
     if ((rc = dense(e, m, L.e_down, m->moe_h, ff, m->moe_y, W, pairs, nullptr, EPI_NONE, 1, &dn))) return rc;
     if (defer) {
-        defer->sel = m->moe_sel; defer->weight = m->moe_weight; defer->pos = tiled ? m->moe_pos : nullptr; defer->rows = m->moe_y; defer->h = in;
+        defer->sel = m->moe_sel; defer->weight = out_weight; defer->pos = tiled ? m->moe_pos : nullptr; defer->rows = m->moe_y; defer->h = in;
         defer->n_experts = d.moe_experts; defer->top = d.moe_top;
         return B2_OK;
     }
     StepProfiler sp(m, st, 7);
-    CK(moe_combine_launch(m->moe_sel, m->moe_weight, tiled ? m->moe_pos : nullptr, m->moe_y, in, d.moe_experts, d.moe_top, W, T, m->oL, st));
+    CK(moe_combine_launch(m->moe_sel, out_weight, tiled ? m->moe_pos : nullptr, m->moe_y, in, d.moe_experts, d.moe_top, W, T, out, st));
     e->launches++;
     return B2_OK;
 }
@@ -1196,10 +1246,10 @@ static int run_mixer(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev&
     }
     return b2_fail(B2_ERR_UNSUPPORTED, "unknown mixer kind");
 }
-static int run_ff(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in, MoeJoinArgs* defer = nullptr) {
-    if (L.d.ff_kind == B2_FF_MOE) return ff_moe(e, m, L, r, in, defer);
-    if (L.d.ff_kind == B2_FF_PIECEWISE) return ff_piecewise(e, m, L, r, in);
-    return L.d.ff_kind == B2_FF_GLU ? ff_glu(e, m, L, r, in) : ff_relu2(e, m, L, r, in);
+static int run_ff(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in, float* out, MoeJoinArgs* defer = nullptr) {
+    if (L.d.ff_kind == B2_FF_MOE) return ff_moe(e, m, L, r, in, out, defer);
+    if (L.d.ff_kind == B2_FF_PIECEWISE) return ff_piecewise(e, m, L, r, in, out);
+    return L.d.ff_kind == B2_FF_GLU ? ff_glu(e, m, L, r, in, out) : ff_relu2(e, m, L, r, in, out);
 }
 
 static int run_layers(b2_engine* e, LayeredModel* m, const RaggedDev& r) {
@@ -1210,7 +1260,9 @@ static int run_layers(b2_engine* e, LayeredModel* m, const RaggedDev& r) {
     int rc;
     {
         StepProfiler sp(m, st, 0);
-        CK(embed_ragged_launch(m->embed.w, m->embed.type, W, r.tok_id, T, m->x, c.embed_scale != 0.f ? c.embed_scale : 1.f, st));
+        BigramTable bg;
+        bg.table = m->bigram.w; bg.w_type = m->bigram.type; bg.buckets = c.bigram_buckets; bg.mul_prev = c.bigram_mul_prev; bg.mul_cur = c.bigram_mul_cur;
+        CK(embed_ragged_launch(m->embed.w, m->embed.type, W, r.tok_id, T, m->x, c.embed_scale != 0.f ? c.embed_scale : 1.f, st, r.tok_prev, &bg));
         e->launches++;
         if (prenorm) {
             CK(resid_rms_norm_launch(m->x, nullptr, 0.f, m->embed_norm, 1.f, 1.f, c.norm_eps, W, T, m->x, st));
@@ -1273,12 +1325,48 @@ static int run_layers(b2_engine* e, LayeredModel* m, const RaggedDev& r) {
             if (d.n_ff > 0) {
                 if ((rc = boundary(L.hc_in[1], L.norm2, m->hn, nullptr, L.canon_w[1], L.canon_state[1], &in))) return rc;
                 const bool moe = d.ff_kind == B2_FF_MOE;
-                if ((rc = run_ff(e, m, L, r, in, moe ? &hj_moe : nullptr))) return rc;
+                if ((rc = run_ff(e, m, L, r, in, m->oL, moe ? &hj_moe : nullptr))) return rc;
                 hj.a = moe ? nullptr : m->oL; hj.mix = L.hc_mix[1]; hj.out = L.hc_out[1];
             }
             if (m->trace || li == c.n_layer - 1) {
                 if ((rc = boundary(nullptr, nullptr, nullptr, m->x, nullptr, nullptr, nullptr))) return rc;
                 if (m->trace) CK(cudaMemcpyAsync(m->trace + ((size_t)li * c.max_step_tokens) * W, m->x, (size_t)T * W * 4, cudaMemcpyDeviceToDevice, st));
+            }
+        }
+        return B2_OK;
+    }
+    if (c.block_style == B2_BLOCK_PARALLEL_LN) {
+        // One kernel per boundary: both outputs of a layer join the stream, and the two norms of the next layer are made from it
+        // (m->hn for the mixer, m->hn2 for the feed-forward block).
+        ParallelJoinArgs pj = {};
+        MoeJoinArgs pj_moe = {};
+        for (int li = 0; li <= c.n_layer; li++) {
+            {
+                StepProfiler sp(m, st, 5);
+                pj.x = m->x; pj.eps = c.norm_eps; pj.moe = pj_moe.sel ? &pj_moe : nullptr;
+                if (li < c.n_layer) {
+                    const LyLayer& L = m->layers[li];
+                    pj.w1 = L.norm1; pj.b1 = L.norm1_b; pj.y1 = m->hn;
+                    if (L.d.n_ff > 0) { pj.w2 = L.norm2; pj.b2 = L.norm2_b; pj.y2 = m->hn2; }
+                }
+                CK(parallel_join_launch(pj, W, T, st));
+                e->launches++;
+                pj = ParallelJoinArgs{}; pj_moe = MoeJoinArgs{};
+            }
+            if (m->trace && li > 0)
+                CK(cudaMemcpyAsync(m->trace + ((size_t)(li - 1) * c.max_step_tokens) * W, m->x, (size_t)T * W * 4, cudaMemcpyDeviceToDevice, st));
+            if (li == c.n_layer) break;
+            LyLayer& L = m->layers[li];
+            if ((rc = run_mixer(e, m, L, r, m->hn))) return rc;
+            pj.a = m->oL;
+            if (L.d.n_ff > 0) {
+                const bool moe = L.d.ff_kind == B2_FF_MOE;
+                if ((rc = run_ff(e, m, L, r, m->hn2, m->oR, moe ? &pj_moe : nullptr))) return rc;
+                if (!moe) pj.b = m->oR;
+                else if (L.d.moe_shared_ff > 0) {
+                    if ((rc = ff_glu(e, m, L, r, m->hn2, m->oR))) return rc;
+                    pj.b = m->oR;
+                }
             }
         }
         return B2_OK;
@@ -1298,10 +1386,10 @@ static int run_layers(b2_engine* e, LayeredModel* m, const RaggedDev& r) {
             if (d.n_ff > 0) {
                 const bool moe = d.ff_kind == B2_FF_MOE;
                 MoeJoinArgs mj = {};
-                if ((rc = run_ff(e, m, L, r, m->x, moe ? &mj : nullptr))) return rc;
+                if ((rc = run_ff(e, m, L, r, m->x, m->oL, moe ? &mj : nullptr))) return rc;
                 const float* dense_part = moe ? nullptr : m->oL;
                 if (moe && d.moe_shared_ff > 0) {          // the shared expert runs for every token; the join adds it to the weighted sum
-                    if ((rc = ff_glu(e, m, L, r, m->x))) return rc;
+                    if ((rc = ff_glu(e, m, L, r, m->x, m->oL))) return rc;
                     dense_part = m->oL;
                 }
                 StepProfiler sp(m, st, 5);
@@ -1315,7 +1403,7 @@ static int run_layers(b2_engine* e, LayeredModel* m, const RaggedDev& r) {
             if (d.n_ff > 0) {
                 if ((rc = join(L.norm2, m->hn))) return rc;
                 const bool moe = d.ff_kind == B2_FF_MOE;
-                if ((rc = run_ff(e, m, L, r, m->hn, moe ? &pending_moe : nullptr))) return rc;
+                if ((rc = run_ff(e, m, L, r, m->hn, m->oL, moe ? &pending_moe : nullptr))) return rc;
                 pending = moe ? nullptr : m->oL;
             }
             if (m->trace || li == c.n_layer - 1) { if ((rc = join(nullptr, nullptr))) return rc; }
@@ -1329,7 +1417,7 @@ static int run_layers(b2_engine* e, LayeredModel* m, const RaggedDev& r) {
                 e->launches++;
             }
             if (d.n_ff > 0) {
-                if ((rc = run_ff(e, m, L, r, m->x))) return rc;
+                if ((rc = run_ff(e, m, L, r, m->x, m->oL))) return rc;
                 StepProfiler sp(m, st, 5);
                 CK(postsum_norm_launch(m->x, m->oL, nullptr, nullptr, nullptr, L.norm2, c.residual_scale, c.norm_eps, W, T, st));
                 e->launches++;
@@ -1372,10 +1460,10 @@ extern "C" int b2_step(b2_engine* e, int n_entries, const int32_t* slots, const 
     CK(cudaSetDevice(c.device));
     cudaStream_t st = e->stream;
     StepChainPdl chain(e->chain_pdl);
-    // ragged description: [tok_id T][tok_seg T][tok_pos T][seg_slot n][seg_start n][seg_len n][seg_pos0 n][tile_seg][tile_row0][rows ...]
+    // ragged description: [tok_id T][tok_seg T][tok_pos T][tok_prev T][seg_slot n][seg_start n][seg_len n][seg_pos0 n][tile_seg][tile_row0][rows ...]
     int* h = m->meta_host;
     const int n = n_entries;
-    int *h_id = h, *h_seg = h + T, *h_pos = h + 2 * T, *h_slot = h + 3 * T, *h_start = h_slot + n, *h_len = h_start + n, *h_p0 = h_len + n;
+    int *h_id = h, *h_seg = h + T, *h_pos = h + 2 * T, *h_prev = h + 3 * T, *h_slot = h + 4 * T, *h_start = h_slot + n, *h_len = h_start + n, *h_p0 = h_len + n;
     int n_tiles = 0;
     for (int i = 0; i < n; i++) n_tiles += (n_tokens[i] + 63) / 64;
     int *h_tseg = h_p0 + n, *h_trow = h_tseg + n_tiles;
@@ -1385,7 +1473,10 @@ extern "C" int b2_step(b2_engine* e, int n_entries, const int32_t* slots, const 
         const int p0 = e->slots[slots[i]].n_past;
         h_slot[i] = slots[i]; h_start[i] = row; h_len[i] = n_tokens[i]; h_p0[i] = p0;
         for (int k = 0; k < n_tokens[i]; k += 64) { h_tseg[tile] = i; h_trow[tile++] = row + k; }
-        for (int k = 0; k < n_tokens[i]; k++, row++) { h_id[row] = tokens[row]; h_seg[row] = i; h_pos[row] = p0 + k; }
+        for (int k = 0; k < n_tokens[i]; k++, row++) {
+            h_id[row] = tokens[row]; h_seg[row] = i; h_pos[row] = p0 + k;
+            h_prev[row] = k > 0 ? tokens[row - 1] : e->slots[slots[i]].last_token;
+        }
     }
     // rows whose logits are needed: the wanted ones, then the last token of every sampled entry
     int n_rows = 0;
@@ -1393,9 +1484,9 @@ extern "C" int b2_step(b2_engine* e, int n_entries, const int32_t* slots, const 
     std::vector<int> samp_row(n, -1);
     for (int i = 0; i < n; i++)
         if (sample && sample[i]) { samp_row[i] = n_rows; h_rows[n_rows++] = h_start[i] + h_len[i] - 1; }
-    const size_t n_meta = (size_t)3 * T + 4 * n + 2 * n_tiles + n_rows;
+    const size_t n_meta = (size_t)4 * T + 4 * n + 2 * n_tiles + n_rows;
     RaggedDev r = {};
-    r.tok_id = m->meta; r.tok_seg = m->meta + T; r.tok_pos = m->meta + 2 * T; r.seg_slot = m->meta + 3 * T;
+    r.tok_id = m->meta; r.tok_seg = m->meta + T; r.tok_pos = m->meta + 2 * T; r.tok_prev = m->meta + 3 * T; r.seg_slot = m->meta + 4 * T;
     r.seg_start = r.seg_slot + n; r.seg_len = r.seg_start + n; r.seg_pos0 = r.seg_len + n; r.T = T; r.n_seg = n;
     r.tile_seg = r.seg_pos0 + n; r.tile_row0 = r.tile_seg + n_tiles; r.n_tiles = n_tiles;
     const int* d_rows = r.tile_row0 + n_tiles;
@@ -1413,7 +1504,7 @@ extern "C" int b2_step(b2_engine* e, int n_entries, const int32_t* slots, const 
             if (c.block_style == B2_BLOCK_OUTNORM_RMS) CK(outnorm_join_launch(nullptr, m->rows, nullptr, m->final_norm, std::max(1, c.norm_groups), c.norm_eps, W, nr, m->rows, st));
             else if (c.block_style == B2_BLOCK_PRENORM_RMS) CK(resid_rms_norm_launch(m->rows, nullptr, 0.f, m->final_norm, 1.f, 1.f, c.norm_eps, W, nr, m->rows, st));
             else if (c.block_style == B2_BLOCK_HYPER_RMS) CK(resid_rms_norm_launch(m->rows, nullptr, 0.f, m->final_norm, 0.f, 1.f, c.norm_eps, W, nr, m->rows, st));
-            else CK(layer_norm_launch(m->rows, m->final_norm, c.norm_eps, W, nr, m->rows, st));
+            else CK(layer_norm_launch(m->rows, m->final_norm, m->final_norm_b, c.norm_eps, W, nr, m->rows, st));
             e->launches += 2;
         }
         DenseArgs hs = {};
@@ -1498,7 +1589,10 @@ extern "C" int b2_step(b2_engine* e, int n_entries, const int32_t* slots, const 
             }
         }
     }
-    for (int i = 0; i < n; i++) e->slots[slots[i]].n_past += n_tokens[i];
+    for (int i = 0; i < n; i++) {
+        e->slots[slots[i]].n_past += n_tokens[i];
+        e->slots[slots[i]].last_token = h_id[h_start[i] + h_len[i] - 1];
+    }
     for (int i = 0; i < n; i++) {
         if (host_sampled) host_sampled[i] = -1;
         if (samp_row[i] >= 0) { if ((rc = b2_sample_enqueue(e, e->slots[slots[i]], i))) return rc; }

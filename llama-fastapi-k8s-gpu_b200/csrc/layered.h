@@ -18,6 +18,7 @@ struct RaggedDev {             // device pointers, valid for one step
     const int* tok_id;         // [T] token ids
     const int* tok_seg;        // [T] segment of each token
     const int* tok_pos;        // [T] position inside its sequence
+    const int* tok_prev;       // [T] the token before it in its sequence (of an earlier step, if need be); -1: it is the first
     const int* seg_slot;       // [n_seg]
     const int* seg_start;      // [n_seg] first row of the segment
     const int* seg_len;        // [n_seg]
@@ -31,10 +32,11 @@ struct RaggedDev {             // device pointers, valid for one step
 // Y[t][n] = epi(sum_k X[t][k] * W[n][k] (+ bias[n])), X f32 [T][ldx], W [N][K] (bf16 or f32), Y f32 [T][ldy].
 // Each output element is one fixed-order sum over k: a row's result does not depend on what else is in the batch.
 // EPI_GLU_SILU: weight rows come in pairs (2i = gate, 2i + 1 = up); output column i = silu(gate) * up, N counts weight rows.
-// EPI_MUL_SIGMOID: the product times sigmoid(aux[t][n]).
+// EPI_GLU_GELU: the same with the tanh form of GELU.
+// EPI_MUL_SIGMOID: the product times sigmoid(aux[t][n]) (aux_one: sigmoid(aux[t][0]) for all columns of a batch entry).
 // EPI_GLU_CLAMP: pairs as above; g = min(gate, p0), u = clamp(up, -p0, p0); output = g * sigmoid(p1 * g) * (u + 1).
 // EPI_PIECEWISE: z > 0: p0 z^2 + z / 2; else p1 (exp(z) - 1 - z) + z / 2.
-enum DenseEpi { EPI_NONE = 0, EPI_BIAS = 1, EPI_BIAS_RELU2 = 2, EPI_GLU_SILU = 3, EPI_MUL_SIGMOID = 4, EPI_GLU_CLAMP = 5, EPI_PIECEWISE = 6 };
+enum DenseEpi { EPI_NONE = 0, EPI_BIAS = 1, EPI_BIAS_RELU2 = 2, EPI_GLU_SILU = 3, EPI_MUL_SIGMOID = 4, EPI_GLU_CLAMP = 5, EPI_PIECEWISE = 6, EPI_GLU_GELU = 7 };
 // Grouped products (mixture of experts): the rows of a step's (token, choice) pairs, each against the matrix of its group.
 //   tiles == nullptr: row p of the product is pair p itself, blockIdx.y walks the pairs one by one (few-token steps);
 //   else: pairs sorted by group, tile i = rows [tile_row0[i], + tile_rows[i]) of group tile_group[i]; *n_tiles of them.
@@ -42,6 +44,7 @@ enum DenseEpi { EPI_NONE = 0, EPI_BIAS = 1, EPI_BIAS_RELU2 = 2, EPI_GLU_SILU = 3
 struct DenseGroups {
     const int* group = nullptr;        // untiled: [rows] group of each row
     const int* x_rows = nullptr;       // [rows] input row of each product row, or null
+    const float* row_scale = nullptr;  // [rows] or null: gate and up of a product row times this before the activation (GLU epilogues)
     const int* tile_group = nullptr;   // tiled: per tile
     const int* tile_row0 = nullptr;
     const int* tile_rows = nullptr;
@@ -63,7 +66,7 @@ struct DenseArgs {
     __nv_bfloat16* xb;              // scratch [T][K] for X rounded to bf16 (large tensor-core steps); null: not available
     float scale = 1.f;              // the product (after the epilogue) times this
     float p0 = 0.f, p1 = 0.f;       // constants of EPI_GLU_CLAMP / EPI_PIECEWISE
-    const float* aux = nullptr; int ldaux = 0;      // EPI_MUL_SIGMOID
+    const float* aux = nullptr; int ldaux = 0; bool aux_one = false;      // EPI_MUL_SIGMOID
     // batch > 1: `batch` independent products, operand b at x + b * x_bs, w + b * w_bs (elements), y + b * y_bs, aux + b * aux_bs
     int batch = 1; long x_bs = 0, w_bs = 0, y_bs = 0, aux_bs = 0;
     int x_span = 0;                 // batch > 1: columns of x that hold all batches' inputs (for the rounded copy), or 0
@@ -72,8 +75,13 @@ struct DenseArgs {
 cudaError_t dense_launch(const DenseArgs& a, cudaStream_t s);
 
 // ---------------------------------------------------------------- mixers and norms (mixers.cu)
-// x[t] = table[tok_id[t]] * scale
-cudaError_t embed_ragged_launch(const void* table, int w_type, int W, const int* tok_id, int T, float* x, float scale, cudaStream_t s);
+// x[t] = table[tok_id[t]] * scale (+ bigram row of (tok_prev[t], tok_id[t]))
+struct BigramTable {           // row (prev * mul_prev + cur * mul_cur) mod buckets; row `buckets` for a sequence's first token
+    const void* table = nullptr; int w_type = 0;
+    int buckets = 0, mul_prev = 0, mul_cur = 0;
+};
+cudaError_t embed_ragged_launch(const void* table, int w_type, int W, const int* tok_id, int T, float* x, float scale, cudaStream_t s,
+                                const int* tok_prev = nullptr, const BigramTable* bigram = nullptr);
 // gather rows: y[i] = x[rows[i]]
 cudaError_t gather_rows_launch(const float* x, int W, const int* rows, int n, float* y, cudaStream_t s);
 
@@ -86,13 +94,14 @@ cudaError_t postsum_norm_launch(float* x, const float* a, const float* wa, const
 // y may be x itself.
 cudaError_t resid_rms_norm_launch(float* x, const float* add, float mult, const float* w, float w_offset, float out_scale,
                                   float eps, int W, int T, float* y, cudaStream_t s);
-// plain layer norm without bias: y[t] = LN(x[t]) * w
-cudaError_t layer_norm_launch(const float* x, const float* w, float eps, int W, int T, float* y, cudaStream_t s);
+// plain layer norm: y[t] = LN(x[t]) * w (+ b)
+cudaError_t layer_norm_launch(const float* x, const float* w, const float* b, float eps, int W, int T, float* y, cudaStream_t s);
 
 struct RotaryTable {           // cos and sin of position * frequency (frequencies already blended, magnitude factor folded
     const float* cos;          // in), [n_ctx][rot_dims / 2] each, built on the host in double precision
     const float* sin;
     int rot_dims;
+    int pairs = 0;             // latent attention: 1 = entries 2i and 2i + 1 are rotated together, 0 = i and i + rot_dims / 2
 };
 struct WindowAttnArgs {
     const float* proj; int ldp; int q_off, k_off;     // projection rows: q at q_off [H*d], k at k_off [G*d]
@@ -206,22 +215,27 @@ cudaError_t group_norm_gate_launch(const GroupNormArgs& a, int T, cudaStream_t s
 // Every token caches one row [c (rank) | rotated shared key part (dr)]; all heads read the same rows. With the per-head
 // key expansion folded into the query (qv[t][h] = [W_uk,h^T q_h | rotated q part]) a head's score is one dot product with
 // the cached row, and the attention output is a weighted sum of the c parts, expanded to values afterwards.
-// Sliding window; the softmax denominator also holds exp(sink[h]).
+// Sliding window; the softmax denominator also holds exp(sink[h]), if there is a sink.
+// Queries come from the input itself (q_off >= 0: the store pass rotates their last dr entries into qv), or through a latent
+// (q_rank > 0: the store pass norms it into cq, the caller expands it into q_raw, whose rotated parts the attention reads).
 struct LatentAttnArgs {
-    const float* proj; int ldp; int q_off, dkv_off;   // q [H][d + dr], dkv [rank + dr]
+    const float* proj; int ldp; int q_off, dkv_off;   // q [H][d + dr], dkv [rank + dr] (dkv_off < 0: the rows are another layer's)
     const float* c_norm_w;                            // [rank]
-    RotaryTable rot;                                  // pairs (i, i + rot_dims / 2)
-    void* pool; int cache_f32;                        // pages [page][block_tokens][rank + dr]
+    int dq_off, q_rank; const float* q_norm_w;        // query latent in the projection row; its norm weight [q_rank]
+    float* cq;                                        // [T][q_rank] normed query latent
+    const float* q_raw;                               // [T][H][d + dr] or null
+    RotaryTable rot;
+    void* pool; int cache_f32; int ld_row;            // pages [page][block_tokens][ld_row], ld_row >= rank + dr
     int* const* block_tables; int block_tokens;
     int H, d, dr, rank, window;
     float scale, eps;
-    const float* sink;                                // [H]
+    const float* sink;                                // [H] or null
     float* qv;                                        // [T][H][rank + dr]; the first `rank` of each head are filled by the caller
     float* o_lat;                                     // [T][H][rank]
     float* split_scratch;      // few-token steps: partial (max, sum, output) per key range, [T][H][splits][rank + 2]
     int split_capacity;        // floats in split_scratch
 };
-// norm of c, rotation of the shared key part, both into the pages; rotated query parts into qv
+// norm of c, rotation of the shared key part, both into the pages; rotated query parts into qv, or norm of the query latent
 cudaError_t latent_store_launch(const LatentAttnArgs& a, const RaggedDev& r, cudaStream_t s);
 cudaError_t latent_attn_launch(const LatentAttnArgs& a, const RaggedDev& r, cudaStream_t s);
 
@@ -233,6 +247,7 @@ struct MoeRouteArgs {
     float scale;
     int mode = 0;                          // 0: weight = softmax over all slots (times scale), `correction` added for the choice only;
                                            // 1: logits + correction choose, weight = softmax over the chosen biased logits
+                                           // 2: as 0 with score = sigmoid of the slot's logit
     int renorm = 0;                        // mode 0: the chosen scores are divided by their sum (+ 1e-20) before the scale
     int* sel; float* weight;               // [T][top]
     int* pair_token;                       // [T][top]: t (the input row of each pair)
@@ -243,6 +258,7 @@ cudaError_t moe_route_launch(const MoeRouteArgs& a, int T, cudaStream_t s);
 struct MoeSortArgs {
     const int* sel; int n_pairs, top, n_experts, tile;      // tile: rows per tile
     int* pos; int* x_rows; int* tile_group; int* tile_row0; int* tile_rows; int* n_tiles; int max_tiles;
+    const float* weight = nullptr; float* row_weight = nullptr;      // weight != null: row_weight[row of pair p] = weight[p]
 };
 cudaError_t moe_sort_launch(const MoeSortArgs& a, cudaStream_t s);
 // out[t] = sum over the token's choices, in choice order, of weight * (expert output row | h[t] for identity slots)
@@ -252,11 +268,21 @@ cudaError_t moe_combine_launch(const int* sel, const float* weight, const int* p
 // the same sum joined to the residual stream in one pass (pre-norm blocks): x[t] += mult * sum; if (y) y[t] = RMS norm of the
 // new x[t] times (w_offset + w). y may be the buffer h points to (a token's h is read before its y is written).
 struct MoeJoinArgs {
-    const int* sel; const float* weight; const int* pos; const float* rows; const float* h;
+    const int* sel; const float* weight; const int* pos; const float* rows; const float* h;     // weight == null: all 1
     int n_experts, top;
 };
 cudaError_t moe_join_launch(const MoeJoinArgs& j, float* x, float mult, const float* w, float w_offset, float eps, int W, int T, float* y,
                             cudaStream_t s);
+
+// Parallel blocks: x[t] += a[t] + (b[t], or a mixture's sum of expert rows); then every norm given, all of the new x[t]:
+// y = (x - mean) / sqrt(var + eps) * w + bias. Any part may be absent (a == b == moe == null: x stays as it is).
+struct ParallelJoinArgs {
+    float* x; const float* a; const float* b; const MoeJoinArgs* moe;
+    const float *w1, *b1; float* y1;
+    const float *w2, *b2; float* y2;
+    float eps;
+};
+cudaError_t parallel_join_launch(const ParallelJoinArgs& a, int W, int T, cudaStream_t s);
 
 // Blocks that norm what a branch RETURNS: v[t] = a[t] (if given) + the mixture's weighted sum (if given); each of `groups` equal
 // consecutive parts of v is brought to unit RMS, the whole is multiplied by w; then x[t] += that (x given) or y[t] = that.

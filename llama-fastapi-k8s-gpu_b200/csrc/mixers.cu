@@ -43,19 +43,34 @@ __device__ __forceinline__ float log_sigmoid_f(float z) { return -softplus_f(-z)
 
 // ---------------------------------------------------------------- embedding, gather
 template <typename TW>
-__global__ void embed_ragged_kernel(const TW* __restrict__ table, int W, const int* __restrict__ tok, float* __restrict__ x, float scale) {
+__global__ void embed_ragged_kernel(const TW* __restrict__ table, int W, const int* __restrict__ tok, float* __restrict__ x, float scale,
+                                    const int* __restrict__ tok_prev, BigramTable bg) {
     griddep_launch();
     griddep_wait();
-    const int t = blockIdx.x;
-    const TW* row = table + (size_t)tok[t] * W;
+    const int t = blockIdx.x, cur = tok[t];
+    const TW* row = table + (size_t)cur * W;
+    size_t pair_row = 0;
+    if (bg.table) {
+        const int prev = tok_prev[t];
+        pair_row = prev < 0 ? bg.buckets : (size_t)(((long long)prev * bg.mul_prev + (long long)cur * bg.mul_cur) % bg.buckets);
+    }
     for (int i = threadIdx.x; i < W; i += blockDim.x) {
-        if constexpr (sizeof(TW) == 2) x[(size_t)t * W + i] = __bfloat162float(row[i]) * scale;
-        else x[(size_t)t * W + i] = row[i] * scale;
+        float v;
+        if constexpr (sizeof(TW) == 2) v = __bfloat162float(row[i]) * scale;
+        else v = row[i] * scale;
+        if (bg.table) {
+            const size_t j = pair_row * W + i;
+            v += bg.w_type == T_BF16 ? __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(bg.table)[j]) : reinterpret_cast<const float*>(bg.table)[j];
+        }
+        x[(size_t)t * W + i] = v;
     }
 }
-cudaError_t embed_ragged_launch(const void* table, int w_type, int W, const int* tok_id, int T, float* x, float scale, cudaStream_t s) {
-    if (w_type == T_BF16) return launch_chain(embed_ragged_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, s, (const __nv_bfloat16*)table, W, tok_id, x, scale);
-    if (w_type == T_F32) return launch_chain(embed_ragged_kernel<float>, dim3(T), dim3(128), 0, s, (const float*)table, W, tok_id, x, scale);
+cudaError_t embed_ragged_launch(const void* table, int w_type, int W, const int* tok_id, int T, float* x, float scale, cudaStream_t s,
+                                const int* tok_prev, const BigramTable* bigram) {
+    const BigramTable bg = bigram ? *bigram : BigramTable{};
+    if (bg.table && !tok_prev) return cudaErrorInvalidValue;
+    if (w_type == T_BF16) return launch_chain(embed_ragged_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, s, (const __nv_bfloat16*)table, W, tok_id, x, scale, tok_prev, bg);
+    if (w_type == T_F32) return launch_chain(embed_ragged_kernel<float>, dim3(T), dim3(128), 0, s, (const float*)table, W, tok_id, x, scale, tok_prev, bg);
     return cudaErrorInvalidValue;
 }
 
@@ -129,8 +144,8 @@ cudaError_t resid_rms_norm_launch(float* x, const float* add, float mult, const 
     return launch_chain(resid_rms_norm_kernel, dim3(T), dim3(256), (size_t)W * 4, s, x, add, mult, w, w_offset, out_scale, eps, W, y);
 }
 
-__global__ void __launch_bounds__(256) layer_norm_kernel(const float* __restrict__ x, const float* __restrict__ w, float eps, int W,
-                                                         float* __restrict__ y) {
+__global__ void __launch_bounds__(256) layer_norm_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ b,
+                                                         float eps, int W, float* __restrict__ y) {
     griddep_launch();
     griddep_wait();
     __shared__ float red[33];
@@ -141,10 +156,61 @@ __global__ void __launch_bounds__(256) layer_norm_kernel(const float* __restrict
     float sq = 0.f;
     for (int i = threadIdx.x; i < W; i += blockDim.x) { const float dlt = x[base + i] - mean; sq += dlt * dlt; }
     const float rstd = 1.f / sqrtf(block_sum(sq, red) / (float)W + eps);
-    for (int i = threadIdx.x; i < W; i += blockDim.x) y[base + i] = (x[base + i] - mean) * rstd * w[i];
+    for (int i = threadIdx.x; i < W; i += blockDim.x) y[base + i] = fmaf((x[base + i] - mean) * rstd, w[i], b ? b[i] : 0.f);
 }
-cudaError_t layer_norm_launch(const float* x, const float* w, float eps, int W, int T, float* y, cudaStream_t s) {
-    return launch_chain(layer_norm_kernel, dim3(T), dim3(256), 0, s, x, w, eps, W, y);
+cudaError_t layer_norm_launch(const float* x, const float* w, const float* b, float eps, int W, int T, float* y, cudaStream_t s) {
+    return launch_chain(layer_norm_kernel, dim3(T), dim3(256), 0, s, x, w, b, eps, W, y);
+}
+
+// parallel blocks: both sublayers' outputs (a mixture's expert rows are summed here) join the 32-bit stream, and both norms of
+// the next layer are made from one mean and one variance; the row lives in shared memory between the passes
+struct ParallelJoinDev { ParallelJoinArgs a; MoeJoinArgs j; int moe; };
+template <int NT>
+__global__ void __launch_bounds__(NT) parallel_join_kernel(ParallelJoinDev p, int W) {
+    griddep_launch();
+    griddep_wait();
+    extern __shared__ float row[];
+    __shared__ float red[33];
+    const ParallelJoinArgs& a = p.a;
+    const MoeJoinArgs& j = p.j;
+    const int t = blockIdx.x;
+    const size_t base = (size_t)t * W;
+    const bool adds = a.a || a.b || p.moe;
+    float sum = 0.f;
+    for (int i = threadIdx.x; i < W; i += NT) {
+        float v = a.x[base + i], y = a.a ? a.a[base + i] : 0.f;
+        if (a.b) y += a.b[base + i];
+        if (p.moe) {
+            float acc = 0.f;
+            for (int c = 0; c < j.top; c++) {
+                const int q = t * j.top + c;
+                const float u = j.sel[q] < j.n_experts ? j.rows[(size_t)(j.pos ? j.pos[q] : q) * W + i] : j.h[base + i];
+                acc = fmaf(j.weight ? j.weight[q] : 1.f, u, acc);
+            }
+            y += acc;
+        }
+        if (adds) { v += y; a.x[base + i] = v; }
+        row[i] = v;
+        sum += v;
+    }
+    if (!a.y1 && !a.y2) return;
+    const float mean = block_sum(sum, red) / (float)W;
+    float sq = 0.f;
+    for (int i = threadIdx.x; i < W; i += NT) { const float dlt = row[i] - mean; sq = fmaf(dlt, dlt, sq); }
+    const float rstd = 1.f / sqrtf(block_sum(sq, red) / (float)W + a.eps);
+    for (int i = threadIdx.x; i < W; i += NT) {
+        const float u = (row[i] - mean) * rstd;
+        if (a.y1) a.y1[base + i] = fmaf(u, a.w1[i], a.b1[i]);
+        if (a.y2) a.y2[base + i] = fmaf(u, a.w2[i], a.b2[i]);
+    }
+}
+cudaError_t parallel_join_launch(const ParallelJoinArgs& a, int W, int T, cudaStream_t s) {
+    ParallelJoinDev p = {};
+    p.a = a;
+    if (a.moe) { p.j = *a.moe; p.moe = 1; }
+    // few tokens: more threads per row, one CTA's latency is all there is
+    if (T <= 16 && W >= 1024) return launch_chain(parallel_join_kernel<1024>, dim3(T), dim3(1024), (size_t)W * 4, s, p, W);
+    return launch_chain(parallel_join_kernel<256>, dim3(T), dim3(256), (size_t)W * 4, s, p, W);
 }
 
 // ---------------------------------------------------------------- window attention

@@ -1,4 +1,4 @@
-// Mixture of experts for the layer-list models: routing (softmax scores, additive choice correction, group-limited
+// Mixture of experts for the layer-list models: routing (softmax or sigmoid scores, additive choice correction, group-limited
 // top-k with identity slots; or biased logits with a softmax over the chosen ones), the bookkeeping that sorts a step's (token, choice) pairs by expert into row tiles for the
 // grouped products of dense.cu, and the weighted combination. Routing arithmetic is 32-bit.
 #include "kernels.h"
@@ -31,13 +31,17 @@ __global__ void __launch_bounds__(32) moe_route_kernel(MoeRouteArgs a) {
     float* gbest = choice + a.n_slots;
     const int t = blockIdx.x, lane = threadIdx.x, n = a.n_slots;
     const float* z = a.logits + (size_t)t * a.ld;
-    float mx = -INFINITY;
-    for (int i = lane; i < n; i += 32) mx = fmaxf(mx, z[i]);
-    mx = warp_max(mx);
-    float sum = 0.f;
-    for (int i = lane; i < n; i += 32) { const float e = expf(z[i] - mx); score[i] = e; sum += e; }
-    sum = warp_sum(sum);
-    for (int i = lane; i < n; i += 32) { const float s = score[i] / sum; score[i] = s; choice[i] = s + (a.correction ? a.correction[i] : 0.f); }
+    if (a.mode == 2) {                             // without a correction the logits choose: the same order, no ties where sigmoid saturates
+        for (int i = lane; i < n; i += 32) { const float s = 1.f / (1.f + expf(-z[i])); score[i] = s; choice[i] = a.correction ? s + a.correction[i] : z[i]; }
+    } else {
+        float mx = -INFINITY;
+        for (int i = lane; i < n; i += 32) mx = fmaxf(mx, z[i]);
+        mx = warp_max(mx);
+        float sum = 0.f;
+        for (int i = lane; i < n; i += 32) { const float e = expf(z[i] - mx); score[i] = e; sum += e; }
+        sum = warp_sum(sum);
+        for (int i = lane; i < n; i += 32) { const float s = score[i] / sum; score[i] = s; choice[i] = s + (a.correction ? a.correction[i] : 0.f); }
+    }
     __syncwarp();
     if (a.n_groups > 1 && a.keep_groups < a.n_groups) {
         const int per = n / a.n_groups;
@@ -158,6 +162,7 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(MoeSortArgs a) {
         if (e >= 0 && e < a.n_experts) {
             row = offset[e] + atomicAdd(&cursor[e], 1);
             a.x_rows[row] = p / a.top;
+            if (a.weight) a.row_weight[row] = a.weight[p];
         }
         a.pos[p] = row;
     }
@@ -179,7 +184,7 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const int* __restrict_
         float acc = 0.f;
         for (int c = 0; c < top; c++) {
             const int p = t * top + c, e = sel[p];
-            const float wv = weight[p];
+            const float wv = weight ? weight[p] : 1.f;
             const float v = e < n_experts ? rows[(size_t)(pos ? pos[p] : p) * W + i] : h[(size_t)t * W + i];
             acc = fmaf(wv, v, acc);
         }
@@ -206,7 +211,7 @@ __global__ void __launch_bounds__(256) moe_join_kernel(MoeJoinArgs j, float* __r
         for (int c = 0; c < j.top; c++) {
             const int p = t * j.top + c, e = j.sel[p];
             const float v = e < j.n_experts ? j.rows[(size_t)(j.pos ? j.pos[p] : p) * W + i] : j.h[base + i];
-            acc = fmaf(j.weight[p], v, acc);
+            acc = fmaf(j.weight ? j.weight[p] : 1.f, v, acc);
         }
         const float v = fmaf(mult, acc, x[base + i]);
         x[base + i] = v;
@@ -245,7 +250,7 @@ __global__ void __launch_bounds__(256) outnorm_join_kernel(float* __restrict__ x
             for (int c = 0; c < j.top; c++) {
                 const int p = t * j.top + c, e = j.sel[p];
                 const float v = e < j.n_experts ? j.rows[(size_t)(j.pos ? j.pos[p] : p) * W + i] : j.h[base + i];
-                acc = fmaf(j.weight[p], v, acc);
+                acc = fmaf(j.weight ? j.weight[p] : 1.f, v, acc);
             }
         row[i] = acc;
     }

@@ -19,9 +19,10 @@ B2_MIX_WINDOW_SCAN, B2_MIX_MATRIX_MEMORY, B2_MIX_LATENT_ATTN, B2_MIX_DELTA_RULE,
 B2_MIX_SINK_DELTA, B2_MIX_SINK_ATTN = 7, 8
 B2_FF_RELU2, B2_FF_MOE, B2_FF_GLU, B2_FF_PIECEWISE = 0, 1, 2, 3
 B2_EXPERT_SILU, B2_EXPERT_CLAMPED = 0, 1
-B2_ATTN_BIAS, B2_ATTN_UNIT_QK, B2_ATTN_TALK, B2_ATTN_HEAD_GATE = 1, 2, 4, 8
-B2_ROUTE_SOFTMAX_ALL, B2_ROUTE_TOPK_SOFTMAX = 0, 1
-B2_BLOCK_POSTSUM_LN, B2_BLOCK_PRENORM_RMS, B2_BLOCK_OUTNORM_RMS, B2_BLOCK_HYPER_RMS = 0, 1, 2, 3
+B2_ACT_SILU, B2_ACT_GELU_TANH = 0, 1
+B2_ATTN_BIAS, B2_ATTN_UNIT_QK, B2_ATTN_TALK, B2_ATTN_HEAD_GATE, B2_ATTN_NO_GATE, B2_ATTN_NO_SINK, B2_ATTN_ROT_PAIRS = 1, 2, 4, 8, 16, 32, 64
+B2_ROUTE_SOFTMAX_ALL, B2_ROUTE_TOPK_SOFTMAX, B2_ROUTE_SIGMOID = 0, 1, 2
+B2_BLOCK_POSTSUM_LN, B2_BLOCK_PRENORM_RMS, B2_BLOCK_OUTNORM_RMS, B2_BLOCK_HYPER_RMS, B2_BLOCK_PARALLEL_LN = 0, 1, 2, 3, 4
 B2_STEP_MAX_ENTRIES = 64
 
 
@@ -42,14 +43,16 @@ class B2LayerDesc(ctypes.Structure):
                                "moe_experts", "moe_identity", "moe_top", "moe_groups", "moe_keep", "pad1_")] + [
         ("moe_scale", c_double), ("moe_route", c_int32), ("moe_shared_ff", c_int32), ("attn_vdim", c_int32), ("pad2_", c_int32),
         ("softcap", c_double), ("branch_scale", c_double * 2)] + [
-        (n, c_int32) for n in ("attn_flags", "weights_of", "moe_expert", "moe_renorm")] + [("moe_limit", c_double), ("moe_alpha", c_double)]
+        (n, c_int32) for n in ("attn_flags", "weights_of", "moe_expert", "moe_renorm")] + [("moe_limit", c_double), ("moe_alpha", c_double)] + [
+        (n, c_int32) for n in ("ff_act", "moe_scale_input", "la_q_rank", "kv_from")]
 
 
 class B2LayeredConfig(ctypes.Structure):
     _fields_ = [(n, c_int32) for n in ("n_layer", "n_embd", "n_vocab")] + [("norm_eps", c_float), ("residual_scale", c_float)] + [
         (n, c_int32) for n in ("n_ctx", "max_seqs", "kv_block_tokens", "kv_num_blocks", "max_step_tokens", "device", "flags",
                                "block_style")] + [("logit_scale", c_float), ("embed_scale", c_float), ("norm_groups", c_int32),
-                                                  ("tie_head", c_int32), ("n_streams", c_int32), ("canon_taps", c_int32)]
+                                                  ("tie_head", c_int32), ("n_streams", c_int32), ("canon_taps", c_int32),
+                                                  ("bigram_buckets", c_int32), ("bigram_mul_prev", c_int32), ("bigram_mul_cur", c_int32)]
 
 
 class B2Sampling(ctypes.Structure):

@@ -35,6 +35,7 @@ class LayeredDims:
     tie_head: bool = False
     n_streams: int = 1
     canon_taps: int = 0
+    bigram: Tuple[int, int, int] = (0, 0, 0)      # buckets (0: none), factors of the previous and the current token, mod buckets
 
 
 def _need(d: dict, key: str, where: str):
