@@ -12,6 +12,7 @@
 #include "quant_blocks.cuh"
 
 #include <algorithm>
+#include <array>
 
 namespace b2 {
 
@@ -61,28 +62,45 @@ __device__ __forceinline__ int x_row(const DenseDev& a, int t) { return (a.group
 
 __device__ __forceinline__ float silu_act(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float gelu_tanh_act(float z) { return 0.5f * z * (1.f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z))); }
+// The epilogue kind is a.epi, or EPI when that is >= 0 (compiled in: the large-tile kernel, where products over a short K are
+// bound by their epilogue).
+template <int EPI>
+__device__ __forceinline__ float epi_value(const DenseDev& a, const float* aux, int t, int n, float v) {
+    const int epi = EPI >= 0 ? EPI : a.epi;
+    if (epi == EPI_BIAS || epi == EPI_BIAS_RELU2) { if (a.bias) v += a.bias[n]; }
+    if (epi == EPI_BIAS_RELU2) { v = fmaxf(v, 0.f); v = v * v; }
+    if (epi == EPI_MUL_SIGMOID) v *= 1.f / (1.f + expf(-aux[(size_t)t * a.ldaux + n * a.aux_ns]));
+    if (epi == EPI_PIECEWISE) v = v > 0.f ? fmaf(a.p0 * v, v, 0.5f * v) : fmaf(a.p1, expm1f(v) - v, 0.5f * v);
+    return v * a.scale;
+}
 // one output column
 __device__ __forceinline__ void epi_store(const DenseDev& a, float* y, const float* aux, int t, int n, float v) {
-    if (a.epi == EPI_BIAS || a.epi == EPI_BIAS_RELU2) { if (a.bias) v += a.bias[n]; }
-    if (a.epi == EPI_BIAS_RELU2) { v = fmaxf(v, 0.f); v = v * v; }
-    if (a.epi == EPI_MUL_SIGMOID) v *= 1.f / (1.f + expf(-aux[(size_t)t * a.ldaux + n * a.aux_ns]));
-    if (a.epi == EPI_PIECEWISE) v = v > 0.f ? fmaf(a.p0 * v, v, 0.5f * v) : fmaf(a.p1, expm1f(v) - v, 0.5f * v);
-    y[(size_t)t * a.ldy + n] = v * a.scale;
+    y[(size_t)t * a.ldy + n] = epi_value<-1>(a, aux, t, n, v);
 }
-// two neighbouring columns n (even) and n + 1; rs: scales of the product rows (GLU epilogues) or null
-__device__ __forceinline__ void epi_store2(const DenseDev& a, float* y, const float* aux, const float* rs, int t, int n, float v0, float v1) {
-    if (rs) { v0 *= rs[t]; v1 *= rs[t]; }
-    if (a.epi == EPI_GLU_SILU || a.epi == EPI_GLU_GELU) {
-        if (n + 1 < a.N) y[(size_t)t * a.ldy + (n >> 1)] = (a.epi == EPI_GLU_SILU ? silu_act(v0) : gelu_tanh_act(v0)) * v1 * a.scale;
+// two neighbouring columns n (even) and n + 1; rs: scales of the product rows (GLU epilogues) or null; vec2: pairs of y are
+// 8-byte aligned
+template <int EPI = -1>
+__device__ __forceinline__ void epi_store2(const DenseDev& a, float* y, const float* aux, const float* rs, int t, int n, float v0, float v1,
+                                           bool vec2 = false) {
+    const int epi = EPI >= 0 ? EPI : a.epi;
+    if (epi == EPI_GLU_SILU || epi == EPI_GLU_GELU || epi == EPI_GLU_CLAMP) {
+        if (n + 1 >= a.N) return;
+        if (rs) { v0 *= rs[t]; v1 *= rs[t]; }
+        float v;
+        if (epi == EPI_GLU_CLAMP) {
+            const float g = fminf(v0, a.p0), u = fminf(fmaxf(v1, -a.p0), a.p0);
+            v = g / (1.f + expf(-a.p1 * g)) * (u + 1.f);
+        } else v = (epi == EPI_GLU_SILU ? silu_act(v0) : gelu_tanh_act(v0)) * v1;
+        y[(size_t)t * a.ldy + (n >> 1)] = v * a.scale;
         return;
     }
-    if (a.epi == EPI_GLU_CLAMP) {
-        const float g = fminf(v0, a.p0), u = fminf(fmaxf(v1, -a.p0), a.p0);
-        if (n + 1 < a.N) y[(size_t)t * a.ldy + (n >> 1)] = g / (1.f + expf(-a.p1 * g)) * (u + 1.f) * a.scale;
+    float* dst = y + (size_t)t * a.ldy + n;
+    if (vec2 && n + 1 < a.N) {
+        *reinterpret_cast<float2*>(dst) = make_float2(epi_value<EPI>(a, aux, t, n, v0), epi_value<EPI>(a, aux, t, n + 1, v1));
         return;
     }
-    if (n < a.N) epi_store(a, y, aux, t, n, v0);
-    if (n + 1 < a.N) epi_store(a, y, aux, t, n + 1, v1);
+    if (n < a.N) dst[0] = epi_value<EPI>(a, aux, t, n, v0);
+    if (n + 1 < a.N) dst[1] = epi_value<EPI>(a, aux, t, n + 1, v1);
 }
 
 // ---------------------------------------------------------------- few tokens: a warp per R weight rows
@@ -356,6 +374,7 @@ __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* smem_s
 
 constexpr int BIG_BM = 128, BIG_BN = 128, BIG_BK = 64, BIG_LD = BIG_BK + 8, BIG_STAGES = 3;
 constexpr int BIG_SMEM = BIG_STAGES * (BIG_BM + BIG_BN) * BIG_LD * 2;
+template <int EPI>
 __global__ void __launch_bounds__(256, 2) dense_mma_big_kernel(const __nv_bfloat16* __restrict__ xb, int ldxb, DenseDev a) {
     griddep_launch();
     griddep_wait();
@@ -421,6 +440,7 @@ __global__ void __launch_bounds__(256, 2) dense_mma_big_kernel(const __nv_bfloat
         }
     }
     const int g = lane >> 2, tq = lane & 3;
+    const bool vec2 = a.ldy % 2 == 0 && (reinterpret_cast<uintptr_t>(y) & 7) == 0;
 #pragma unroll
     for (int mi = 0; mi < 4; mi++)
 #pragma unroll
@@ -428,7 +448,7 @@ __global__ void __launch_bounds__(256, 2) dense_mma_big_kernel(const __nv_bfloat
 #pragma unroll
             for (int e = 0; e < 4; e += 2) {
                 const int t = t0 + wm + mi * 16 + g + (e >> 1) * 8;
-                if (t < T) epi_store2(a, y, aux, a.g.row_scale, t, n0 + wn + ni * 8 + 2 * tq, acc[mi][ni][e], acc[mi][ni][e + 1]);
+                if (t < T) epi_store2<EPI>(a, y, aux, a.g.row_scale, t, n0 + wn + ni * 8 + 2 * tq, acc[mi][ni][e], acc[mi][ni][e + 1], vec2);
             }
 }
 
@@ -465,14 +485,20 @@ cudaError_t dense_launch(const DenseArgs& a, cudaStream_t s) {
                         (a.batch == 1 || (a.x_span > 0 && a.x_bs % 8 == 0 && a.w_bs % 8 == 0));
     if (d.grouped == 2 && a.groups->tile_max == BIG_BM && !big_ok) return cudaErrorInvalidValue;
     if (big_ok && (d.grouped ? a.groups->tile_max == BIG_BM : a.T >= 64)) {
-        static bool attr_done = false;
-        if (!attr_done) { cudaFuncSetAttribute(dense_mma_big_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, BIG_SMEM); attr_done = true; }
+        static const auto kernels = [] {
+            std::array<void (*)(const __nv_bfloat16*, int, DenseDev), 8> k = {
+                dense_mma_big_kernel<EPI_NONE>, dense_mma_big_kernel<EPI_BIAS>, dense_mma_big_kernel<EPI_BIAS_RELU2>, dense_mma_big_kernel<EPI_GLU_SILU>,
+                dense_mma_big_kernel<EPI_MUL_SIGMOID>, dense_mma_big_kernel<EPI_GLU_CLAMP>, dense_mma_big_kernel<EPI_PIECEWISE>, dense_mma_big_kernel<EPI_GLU_GELU>};
+            for (auto f : k) cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, BIG_SMEM);
+            return k;
+        }();
+        if (a.epi < 0 || a.epi >= (int)kernels.size()) return cudaErrorInvalidValue;
         const long pairs = (long)x_rows_total * (span / 2);
         cudaError_t ce = launch_chain(rows_to_bf16_kernel, dim3((unsigned)std::min<long>((pairs + 255) / 256, 148 * 8)), dim3(256), 0, s,
                                       a.x, a.ldx, x_rows_total, span, a.xb);
         if (ce != cudaSuccess) return ce;
         const unsigned gy = d.grouped ? (unsigned)a.groups->max_tiles : (unsigned)((a.T + BIG_BM - 1) / BIG_BM);
-        return launch_chain(dense_mma_big_kernel, dim3((a.N + BIG_BN - 1) / BIG_BN, gy, gz), dim3(256), (size_t)BIG_SMEM, s,
+        return launch_chain(kernels[a.epi], dim3((a.N + BIG_BN - 1) / BIG_BN, gy, gz), dim3(256), (size_t)BIG_SMEM, s,
                             (const __nv_bfloat16*)a.xb, span, d);
     }
     dim3 grid((a.N + 63) / 64, d.grouped ? (unsigned)a.groups->max_tiles : (unsigned)((a.T + 63) / 64), gz);
