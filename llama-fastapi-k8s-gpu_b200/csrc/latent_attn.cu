@@ -42,11 +42,11 @@ __device__ __forceinline__ float query_at(const LatentAttnArgs& a, int t, int h,
 }
 }  // namespace
 
-// grid (T), 128 threads
-__global__ void __launch_bounds__(128) latent_store_kernel(LatentAttnArgs a, RaggedDev r) {
+// grid (T), 128 threads (few-token steps: 512, a row's latency is all there is)
+__global__ void __launch_bounds__(512) latent_store_kernel(LatentAttnArgs a, RaggedDev r) {
     griddep_launch();
     griddep_wait();
-    __shared__ float red[2][4];
+    __shared__ float red[2][16];
     const int t = blockIdx.x, pos = r.tok_pos[t];
     const int slot = r.seg_slot[r.tok_seg[t]];
     const int Dk = a.rank + a.dr;
@@ -59,14 +59,16 @@ __global__ void __launch_bounds__(128) latent_store_kernel(LatentAttnArgs a, Rag
     ss = warp_sum(ss); sq = warp_sum(sq);
     if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = ss; red[1][threadIdx.x >> 5] = sq; }
     __syncthreads();
+    float ss_all = 0.f, sq_all = 0.f;
+    for (int k = 0; k < (int)blockDim.x / 32; k++) { ss_all += red[0][k]; sq_all += red[1][k]; }
     if (own) {
         const size_t dst = ((size_t)a.block_tables[slot][pos / a.block_tokens] * a.block_tokens + pos % a.block_tokens) * a.ld_row;
-        const float rinv = 1.f / sqrtf((red[0][0] + red[0][1] + red[0][2] + red[0][3]) / (float)a.rank + a.eps);
+        const float rinv = 1.f / sqrtf(ss_all / (float)a.rank + a.eps);
         for (int i = threadIdx.x; i < a.rank; i += blockDim.x) row_store(a.pool, a.cache_f32, dst + i, dkv[i] * rinv * a.c_norm_w[i]);
         for (int i = threadIdx.x; i < a.dr; i += blockDim.x) row_store(a.pool, a.cache_f32, dst + a.rank + i, rotated_at(dkv + a.rank, i, pos, a.rot));
     }
     if (a.q_rank > 0) {
-        const float rinv = 1.f / sqrtf((red[1][0] + red[1][1] + red[1][2] + red[1][3]) / (float)a.q_rank + a.eps);
+        const float rinv = 1.f / sqrtf(sq_all / (float)a.q_rank + a.eps);
         for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) a.cq[(size_t)t * a.q_rank + i] = dq[i] * rinv * a.q_norm_w[i];
         return;
     }
@@ -77,7 +79,7 @@ __global__ void __launch_bounds__(128) latent_store_kernel(LatentAttnArgs a, Rag
     }
 }
 cudaError_t latent_store_launch(const LatentAttnArgs& a, const RaggedDev& r, cudaStream_t s) {
-    return launch_chain(latent_store_kernel, dim3(r.T), dim3(128), 0, s, a, r);
+    return launch_chain(latent_store_kernel, dim3(r.T), dim3(r.T <= 8 ? 512 : 128), 0, s, a, r);
 }
 
 // grid (T, H, splits), 8 warps: CTA z takes the z-th range of the visible keys, warp w its keys w, w + 8, ...; a lane holds
@@ -240,21 +242,30 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_pairs_kernel(Latent
     }
 }
 
-// sum of the key ranges of one (token, head) in range order (some range has keys, so the sum is never empty)
+// sum of the key ranges of one (token, head) in range order (some range has keys, so the sum is never empty); at most 32 ranges,
+// one lane each for the weights. grid (T, H, chunks of 128 latent columns)
+constexpr int LA_MAX_SPLITS = 16;
 __global__ void __launch_bounds__(128) latent_merge_kernel(LatentAttnArgs a, int n_splits) {
     griddep_launch();
     griddep_wait();
-    const int t = blockIdx.x, h = blockIdx.y, n = a.rank + 2;
+    __shared__ float weight[32];
+    const int t = blockIdx.x, h = blockIdx.y, n = a.rank + 2, i = blockIdx.z * 128 + threadIdx.x;
     const float* part = a.split_scratch + ((size_t)t * a.H + h) * n_splits * n;
-    float M = -INFINITY;
-    for (int s2 = 0; s2 < n_splits; s2++) M = fmaxf(M, part[(size_t)s2 * n]);
-    float L = 0.f;
-    for (int s2 = 0; s2 < n_splits; s2++) { const float ms = part[(size_t)s2 * n]; if (ms > -INFINITY) L += part[(size_t)s2 * n + 1] * expf(ms - M); }
-    for (int i = threadIdx.x; i < a.rank; i += blockDim.x) {
-        float o = 0.f;
-        for (int s2 = 0; s2 < n_splits; s2++) { const float ms = part[(size_t)s2 * n]; if (ms > -INFINITY) o += part[(size_t)s2 * n + 2 + i] * expf(ms - M); }
-        a.o_lat[((size_t)t * a.H + h) * a.rank + i] = o / L;
+    float v[LA_MAX_SPLITS];
+#pragma unroll
+    for (int s2 = 0; s2 < LA_MAX_SPLITS; s2++) v[s2] = s2 < n_splits && i < a.rank ? part[(size_t)s2 * n + 2 + i] : 0.f;
+    if (threadIdx.x < 32) {
+        const bool on = threadIdx.x < n_splits;
+        const float m = on ? part[(size_t)threadIdx.x * n] : -INFINITY, l = on ? part[(size_t)threadIdx.x * n + 1] : 0.f;
+        const float w = expf(m - warp_max(m));            // an empty range: 0
+        weight[threadIdx.x] = w / warp_sum(w * l);
     }
+    __syncthreads();
+    if (i >= a.rank) return;
+    float o = 0.f;
+#pragma unroll
+    for (int s2 = 0; s2 < LA_MAX_SPLITS; s2++) if (s2 < n_splits) o = fmaf(v[s2], weight[s2], o);
+    a.o_lat[((size_t)t * a.H + h) * a.rank + i] = o;
 }
 
 // Tensor-core prompt kernel (bf16 pages, rank and rank + dr multiples of 16): a CTA takes one tile of up to 64 consecutive
@@ -425,7 +436,7 @@ cudaError_t latent_attn_launch(const LatentAttnArgs& a, const RaggedDev& r, cuda
     // a step of a few tokens does not fill the GPU with one CTA per (token, head): split the keys (up to 16 ranges)
     int splits = 1;
     if (a.split_scratch && r.T * a.H < 148) {
-        splits = std::min({16, (2 * 148) / (r.T * a.H), std::max(1, a.window / 32)});
+        splits = std::min({LA_MAX_SPLITS, (2 * 148) / (r.T * a.H), std::max(1, a.window / 32)});
         while (splits > 1 && (size_t)r.T * a.H * splits * (a.rank + 2) > (size_t)a.split_capacity) splits--;
     }
     const dim3 grid(r.T, a.H, splits), block(LA_WARPS * 32);
@@ -442,7 +453,7 @@ cudaError_t latent_attn_launch(const LatentAttnArgs& a, const RaggedDev& r, cuda
     else if (Dk <= 320) ce = launch_chain(latent_attn_kernel<10>, grid, block, smem, s, a, r);
     else ce = launch_chain(latent_attn_kernel<20>, grid, block, smem, s, a, r);
     if (ce != cudaSuccess || splits == 1) return ce;
-    return launch_chain(latent_merge_kernel, dim3(r.T, a.H), dim3(128), 0, s, a, splits);
+    return launch_chain(latent_merge_kernel, dim3(r.T, a.H, (a.rank + 127) / 128), dim3(128), 0, s, a, splits);
 }
 
 }  // namespace b2
