@@ -153,7 +153,8 @@ int b2_synchronize(b2_engine* e);
                                     rotate-half rotation, the heads' weights mixed across heads, one sigmoid gate per head) beside a
                                     gated delta rule with ONE input-dependent decay per head; the two outputs are RMS-normed over the
                                     width and averaged */
-#define B2_MIX_SINK_ATTN 8       /* the same softmax attention alone; what differs is chosen by attn_flags */
+#define B2_MIX_SINK_ATTN 8       /* the same softmax attention alone; what differs is chosen by attn_flags (sink, gate, biases, norms,
+                                    convolutions) and by softcap, qtemp_* */
 #define B2_FF_RELU2 0            /* squared-ReLU block with biases (when n_ff > 0) */
 #define B2_FF_MOE 1              /* routed mixture of gated (SiLU) experts, n_ff = width of one expert */
 #define B2_FF_GLU 2              /* gated unit without biases: down(act(gate x) * (up x)), act = ff_act */
@@ -162,17 +163,26 @@ int b2_synchronize(b2_engine* e);
 #define B2_ACT_SILU 0            /* ff_act: z * sigmoid(z) */
 #define B2_ACT_GELU_TANH 1       /* ff_act: z / 2 * (1 + tanh(sqrt(2 / pi) * (z + 0.044715 z^3))) */
 #define B2_EXPERT_SILU 0         /* expert: down(silu(gate x) * (up x)) */
+#define B2_EXPERT_RELU2 2        /* expert: down(relu(up x)^2), no gate */
 #define B2_EXPERT_CLAMPED 1      /* expert: g = min(gate x, limit), u = clamp(up x, -limit, limit); down(g * sigmoid(alpha g) * (u + 1)) */
 #define B2_ATTN_BIAS 1           /* attn_flags: q, k, v projections carry biases (tensors q.b, k.b, v.b) */
 #define B2_ATTN_UNIT_QK 2        /* after the rotation every head's q and k are divided by their RMS (no weight) */
 #define B2_ATTN_TALK 4           /* weight_h(i, j) <- sum_g talk[h][g] weight_g(i, j) after the softmax (tensor talk [H][H]) */
 #define B2_ATTN_HEAD_GATE 8      /* the sigmoid output gate is one number per head (tensor g [H][W]); else one per output entry */
-#define B2_ATTN_NO_GATE 16       /* latent attention: no output gate (no tensor g) */
-#define B2_ATTN_NO_SINK 32       /* latent attention: ordinary softmax (no tensor sink) */
+#define B2_ATTN_NO_GATE 16       /* no output gate (no tensor g) */
+#define B2_ATTN_NO_SINK 32       /* ordinary softmax (no tensor sink) */
 #define B2_ATTN_ROT_PAIRS 64     /* latent attention: entries 2i and 2i + 1 are rotated together; else i and i + rot_dims / 2 */
+#define B2_ATTN_CONV 128         /* softmax attention: q, k and v each pass a causal convolution of conv_taps taps right after the
+                                    projection, no bias, no activation (tensors q.conv, k.conv, v.conv [channels][taps]) */
+#define B2_ATTN_FULL_NORM 256    /* softmax attention: q and k are RMS-normed over the whole projection, all heads at once (tensors
+                                    q.norm, k.norm of that size) */
+#define B2_ATTN_UNIT_SINK 512    /* softmax attention: one is added to every denominator (a sink with score 0; no tensor) */
+#define B2_ATTN_OUT_BIAS 1024    /* softmax attention: the output projection has a bias (tensor o.b) */
 #define B2_ROUTE_SOFTMAX_ALL 0   /* scores = softmax over all slots; an additive correction steers the choice only */
 #define B2_ROUTE_TOPK_SOFTMAX 1  /* biased logits choose; weights = softmax over the chosen logits */
 #define B2_ROUTE_SIGMOID 2       /* scores = sigmoid of each logit; the largest (+ correction, if any) are chosen */
+#define B2_ROUTE_TABLE 3         /* no router: tensor mlp.table [n_vocab][moe_top] (I32) gives every token id its experts, each with
+                                    weight 1 / moe_top */
 #define B2_BLOCK_POSTSUM_LN 0    /* x <- LayerNorm(alpha * x + f(x)) */
 #define B2_BLOCK_PRENORM_RMS 1   /* x <- x + m * f(RMSNorm(x) * (1 + w)); the embedding and the output are normed the same way */
 #define B2_BLOCK_OUTNORM_RMS 2   /* x <- x + RMSNorm_parts(f(x)) * w: the branch OUTPUT is normed, over norm_groups equal parts;
@@ -184,6 +194,8 @@ int b2_synchronize(b2_engine* e);
                                     The output norm reads the sum of the copies. */
 #define B2_BLOCK_PARALLEL_LN 4   /* x <- x + (mixer(LN1(x)) + ff(LN2(x))), both of the same x; LN with weight and bias (tensors norm1,
                                     norm1.b, ...); the output norm has the same form */
+#define B2_BLOCK_PARALLEL_ONE_LN 5  /* x <- x + (mixer(n) + ff(n)), n = LN(x) * w, one norm for both and no bias (tensor norm1); the output
+                                    norm has the same form */
 typedef struct b2_layer_desc {
     int32_t mixer;            /* B2_MIX_* */
     int32_t n_ff;             /* width of the feed-forward block (of one expert for B2_FF_MOE); 0 = the layer has none */
@@ -226,6 +238,11 @@ typedef struct b2_layer_desc {
                                  input by one map (tensor q) */
     int32_t kv_from;          /* latent attention: 1 + index of the earlier layer whose cached rows this one reads (it has no dkv of
                                  its own); 0: its own */
+    int32_t loop_pass;        /* 1 + number t of the pass over a repeated run of layers that starts ahead of this entry (0: none starts):
+                                 x <- loop.in [x; x0] + loop.step[t], x0 = the embedding output (tensors loop.in [n_embd][2 n_embd],
+                                 loop.step [loop_times][n_embd]) */
+    int32_t moe_shared_gate;  /* != 0: the shared expert's output times sigmoid(shared.sg x), one number per token */
+    double qtemp_coef, qtemp_every;      /* softmax attention: q at position p times 1 + coef ln(floor((p + 1) / every) + 1); coef 0: off */
 } b2_layer_desc;
 typedef struct b2_layered_config {
     int32_t n_layer, n_embd, n_vocab;
@@ -245,6 +262,8 @@ typedef struct b2_layered_config {
     /* bigram embedding: the row (previous token * mul_prev + token * mul_cur) mod buckets of tensor "bigram" [buckets + 1] is added to
      * the embedding row; a sequence's first token takes row `buckets`. 0 buckets: none. The factors are given mod buckets. */
     int32_t bigram_buckets, bigram_mul_prev, bigram_mul_cur;
+    int32_t embed_sinusoid;   /* != 0: entry 2i of the embedding output gets sin(p 10000^(-2i / n_embd)) added, entry 2i + 1 the cos */
+    int32_t loop_times;       /* rows of tensor loop.step (0: no entry has a loop_pass) */
 } b2_layered_config;
 /* Then b2_upload_tensor for every tensor (BF16 / F32), b2_engine_finalize, b2_seq_set_blocks / b2_seq_begin (n_past must be
  * 0: recurrent state cannot be rewound; it zeroes the slot's state) as for any engine. */

@@ -26,6 +26,7 @@ struct DenseDev {
     const float* bias;
     float* y; int ldy;
     int T, N, K, epi;
+    int n_act;                     // EPI_BIAS_TAIL_RELU2: first column of the tail
     float scale, p0, p1;
     const float* aux; int ldaux, aux_ns;      // aux column of output column n: n * aux_ns
     long x_bs, w_bs, y_bs, aux_bs;
@@ -67,8 +68,8 @@ __device__ __forceinline__ float gelu_tanh_act(float z) { return 0.5f * z * (1.f
 template <int EPI>
 __device__ __forceinline__ float epi_value(const DenseDev& a, const float* aux, int t, int n, float v) {
     const int epi = EPI >= 0 ? EPI : a.epi;
-    if (epi == EPI_BIAS || epi == EPI_BIAS_RELU2) { if (a.bias) v += a.bias[n]; }
-    if (epi == EPI_BIAS_RELU2) { v = fmaxf(v, 0.f); v = v * v; }
+    if (epi == EPI_BIAS || epi == EPI_BIAS_RELU2 || epi == EPI_BIAS_TAIL_RELU2) { if (a.bias) v += a.bias[n]; }
+    if (epi == EPI_BIAS_RELU2 || (epi == EPI_BIAS_TAIL_RELU2 && n >= a.n_act)) { v = fmaxf(v, 0.f); v = v * v; }
     if (epi == EPI_MUL_SIGMOID) v *= 1.f / (1.f + expf(-aux[(size_t)t * a.ldaux + n * a.aux_ns]));
     if (epi == EPI_PIECEWISE) v = v > 0.f ? fmaf(a.p0 * v, v, 0.5f * v) : fmaf(a.p1, expm1f(v) - v, 0.5f * v);
     return v * a.scale;
@@ -460,7 +461,7 @@ cudaError_t dense_launch(const DenseArgs& a, cudaStream_t s) {
     const bool wb = a.w_type == T_BF16;
     DenseDev d = {};
     d.x = a.x; d.ldx = a.ldx; d.w = a.w; d.bias = a.bias; d.y = a.y; d.ldy = a.ldy; d.T = a.T; d.N = a.N; d.K = a.K; d.epi = a.epi;
-    d.scale = a.scale; d.p0 = a.p0; d.p1 = a.p1; d.aux = a.aux; d.ldaux = a.ldaux; d.aux_ns = a.aux_one ? 0 : 1; d.x_bs = a.x_bs; d.w_bs = a.w_bs; d.y_bs = a.y_bs; d.aux_bs = a.aux_bs;
+    d.n_act = a.n_act; d.scale = a.scale; d.p0 = a.p0; d.p1 = a.p1; d.aux = a.aux; d.ldaux = a.ldaux; d.aux_ns = a.aux_one ? 0 : 1; d.x_bs = a.x_bs; d.w_bs = a.w_bs; d.y_bs = a.y_bs; d.aux_bs = a.aux_bs;
     if (a.groups) { d.g = *a.groups; d.grouped = a.groups->tile_group ? 2 : 1; }
     if (d.grouped == 1 || (!d.grouped && a.T <= ROWS_MAX_T)) return wb ? launch_rows<__nv_bfloat16>(d, a.batch, s) : launch_rows<float>(d, a.batch, s);
     // few output columns in 32-bit (router scores): the tiled kernel would run a handful of CTAs over the whole K; the
@@ -486,9 +487,10 @@ cudaError_t dense_launch(const DenseArgs& a, cudaStream_t s) {
     if (d.grouped == 2 && a.groups->tile_max == BIG_BM && !big_ok) return cudaErrorInvalidValue;
     if (big_ok && (d.grouped ? a.groups->tile_max == BIG_BM : a.T >= 64)) {
         static const auto kernels = [] {
-            std::array<void (*)(const __nv_bfloat16*, int, DenseDev), 8> k = {
+            std::array<void (*)(const __nv_bfloat16*, int, DenseDev), 9> k = {
                 dense_mma_big_kernel<EPI_NONE>, dense_mma_big_kernel<EPI_BIAS>, dense_mma_big_kernel<EPI_BIAS_RELU2>, dense_mma_big_kernel<EPI_GLU_SILU>,
-                dense_mma_big_kernel<EPI_MUL_SIGMOID>, dense_mma_big_kernel<EPI_GLU_CLAMP>, dense_mma_big_kernel<EPI_PIECEWISE>, dense_mma_big_kernel<EPI_GLU_GELU>};
+                dense_mma_big_kernel<EPI_MUL_SIGMOID>, dense_mma_big_kernel<EPI_GLU_CLAMP>, dense_mma_big_kernel<EPI_PIECEWISE>, dense_mma_big_kernel<EPI_GLU_GELU>,
+                dense_mma_big_kernel<EPI_BIAS_TAIL_RELU2>};
             for (auto f : k) cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, BIG_SMEM);
             return k;
         }();

@@ -3,11 +3,12 @@
 // scan, an mLSTM matrix memory, latent attention, the gated delta rule, a Mamba-2 state-space layer, chunk-local sigmoid
 // attention beside fixed-decay linear attention, softmax attention with a sink alone or beside a head-decay delta rule.
 // Feed-forward blocks: squared ReLU with biases, a gated SiLU or GELU unit, a block with a piecewise activation, or a routed
-// mixture of gated experts (SiLU or clamped; with an optional shared expert). Five block styles: layer norm AFTER each residual
+// mixture of experts (gated SiLU, clamped, or ungated squared ReLU; chosen by scores or by a table of token ids; with an optional
+// shared expert). Six block styles: layer norm AFTER each residual
 // sum, pre-norm (zero-centred RMS weights) with a scaled branch, an RMS norm in parts on each branch's OUTPUT, pre-norm over
 // several copies of the stream with mixing matrices and a convolution on every sublayer's input, or parallel sublayers behind two
-// layer norms of the same stream. A layer entry may name another layer's tensors (a repeated run of layers: shared weights, cache
-// and state of its own); a latent-attention layer may read the rows another layer caches. Shares the engine object with the
+// layer norms of the same stream or behind one. A layer entry may name another layer's tensors (a repeated run of layers: shared weights, cache
+// and state of its own; a pass over such a run may start with a map of the stream and the embedding output); a latent-attention layer may read the rows another layer caches. Shares the engine object with the
 // llama graph (engine.cu): tensors, sequence slots and their page tables, sampler state, stream, error reporting. Owns: fused
 // projection matrices, per-layer cache pages, per-slot recurrent state, the step workspace.
 #include "engine_state.h"
@@ -68,7 +69,12 @@ struct LyLayer {
     // | b | a | g); reuses attn_o, sink, left_w, right_w, rot_*, k_pool, v_pool and the delta rule's st_* fields
     DenseW sk_proj;
     int gl_off = 0, ra_off = 0, rg_off = 0;
-    float *sk_bias = nullptr, *talk = nullptr;
+    float *sk_bias = nullptr, *talk = nullptr, *o_bias = nullptr;
+    // blocks behind one norm: the shared expert's gate and up rows ride at the end of sk_proj (| sg | up), its down map beside attn_o's
+    // columns: both sublayers read the same row, and one product maps the heads' outputs and the gated hidden row together
+    int sg_off = -1, su_off = -1;
+    // experts by token id: this layer's part of the step's plan
+    MoeTableLayer plan = {};
     // several copies of the stream: per sublayer (0 mixer, 1 feed-forward) read weights, mixing matrix, write weights; the
     // convolution on the sublayer's input and the last taps-1 inputs per slot
     float *hc_in[2] = {}, *hc_mix[2] = {}, *hc_out[2] = {}, *canon_w[2] = {}, *canon_state[2] = {};
@@ -81,7 +87,12 @@ struct LayeredModel {
     b2_layered_config c = {};
     std::vector<LyLayer> layers;
     std::vector<void*> owned;          // device allocations freed at destroy
-    DenseW embed, head, bigram;
+    DenseW embed, head, bigram, loop_in;
+    float* loop_step = nullptr;        // [loop_times][W]
+    float* loop_x = nullptr;           // [max_step_tokens][2 W]: stream | embedding output, the input of loop_in
+    double* turns = nullptr;           // position sinusoid: turns per position of each pair
+    MoeTableLayer* table_layers = nullptr;      // device: plans of the layers whose experts are chosen by token id
+    int n_table = 0, table_experts = 0;
     float *final_norm = nullptr, *final_norm_b = nullptr, *embed_norm = nullptr;
     bool exact = false;                // B2_FLAG_F32
     int** block_tables = nullptr;      // device [max_seqs] -> page table
@@ -136,6 +147,20 @@ static int find(b2_engine* e, const std::string& name, int64_t ne0, int64_t ne1,
                                        "], expected [" + std::to_string(ne1) + "," + std::to_string(ne0) + "]");
     if (t.type != T_BF16 && t.type != T_F32) return b2_fail(B2_ERR_UNSUPPORTED, "tensor " + name + " must be BF16 or F32");
     out = t;
+    return B2_OK;
+}
+
+// an integer table, every entry in [0, limit)
+static int int_table(b2_engine* e, const std::string& name, int64_t rows, int64_t cols, int limit, const int** out) {
+    auto it = e->tensors.find(name);
+    if (it == e->tensors.end()) return b2_fail(B2_ERR_STATE, "missing tensor " + name);
+    const DevTensor& t = it->second;
+    if (t.ne0 != cols || t.ne1 != rows || t.type != T_I32)
+        return b2_fail(B2_ERR_ARG, "tensor " + name + " must be I32 of shape [" + std::to_string(rows) + "," + std::to_string(cols) + "]");
+    std::vector<int> host((size_t)(rows * cols));
+    CK(cudaMemcpy(host.data(), t.ptr, host.size() * 4, cudaMemcpyDeviceToHost));
+    for (int v : host) if (v < 0 || v >= limit) return b2_fail(B2_ERR_ARG, "tensor " + name + ": entry " + std::to_string(v) + " is no expert");
+    *out = reinterpret_cast<const int*>(t.ptr);
     return B2_OK;
 }
 
@@ -204,31 +229,46 @@ static int concat_f32(b2_engine* e, LayeredModel* m, const std::vector<std::pair
     return B2_OK;
 }
 
-// the experts of a layer stacked: [E][2 ff][W] with gate and up rows interleaved, and [E][W][ff]
+// the experts of a layer stacked: [E][2 ff][W] with gate and up rows interleaved (gated) or [E][ff][W], and [E][W][ff]
 // (names p + "<index>."); n_experts == 0: the single unit named p + "."
-static int stack_experts(b2_engine* e, LayeredModel* m, const std::string& p, int n_experts, int ff, int W, DenseW& gate_up, DenseW& down) {
+static int stack_experts(b2_engine* e, LayeredModel* m, const std::string& p, int n_experts, int ff, int W, DenseW& up, DenseW& down, bool gated = true) {
     int type = -1;
     void *gu = nullptr, *dn = nullptr;
-    const int E = std::max(1, n_experts);
+    const int E = std::max(1, n_experts), per = gated ? 2 : 1;
     for (int x = 0; x < E; x++) {
         DevTensor tg, tu, td;
         const std::string q = n_experts > 0 ? p + std::to_string(x) + "." : p + ".";
         int rc;
-        if ((rc = find(e, q + "gate", W, ff, tg)) || (rc = find(e, q + "up", W, ff, tu)) || (rc = find(e, q + "down", ff, W, td))) return rc;
+        if ((gated && (rc = find(e, q + "gate", W, ff, tg))) || (rc = find(e, q + "up", W, ff, tu)) || (rc = find(e, q + "down", ff, W, td))) return rc;
         if (type < 0) {
-            type = tg.type;
+            type = tu.type;
             const size_t esz = type == T_BF16 ? 2 : 4;
-            if ((rc = dev_alloc(m, &gu, (size_t)E * 2 * ff * W * esz + 64)) || (rc = dev_alloc(m, &dn, (size_t)E * W * ff * esz + 64))) return rc;
+            if ((rc = dev_alloc(m, &gu, (size_t)E * per * ff * W * esz + 64)) || (rc = dev_alloc(m, &dn, (size_t)E * W * ff * esz + 64))) return rc;
         }
-        if (tg.type != type || tu.type != type || td.type != type) return b2_fail(B2_ERR_UNSUPPORTED, q + ": the experts of a layer must share a dtype");
+        if ((gated && tg.type != type) || tu.type != type || td.type != type) return b2_fail(B2_ERR_UNSUPPORTED, q + ": the experts of a layer must share a dtype");
         const size_t esz = type == T_BF16 ? 2 : 4, rowb = (size_t)W * esz;
-        char* base = (char*)gu + (size_t)x * 2 * ff * rowb;
-        CK(cudaMemcpy2DAsync(base, 2 * rowb, tg.ptr, rowb, rowb, ff, cudaMemcpyDeviceToDevice, e->stream));
-        CK(cudaMemcpy2DAsync(base + rowb, 2 * rowb, tu.ptr, rowb, rowb, ff, cudaMemcpyDeviceToDevice, e->stream));
+        char* base = (char*)gu + (size_t)x * per * ff * rowb;
+        if (gated) CK(cudaMemcpy2DAsync(base, 2 * rowb, tg.ptr, rowb, rowb, ff, cudaMemcpyDeviceToDevice, e->stream));
+        CK(cudaMemcpy2DAsync(base + (per - 1) * rowb, per * rowb, tu.ptr, rowb, rowb, ff, cudaMemcpyDeviceToDevice, e->stream));
         CK(cudaMemcpyAsync((char*)dn + (size_t)x * W * ff * esz, td.ptr, (size_t)W * ff * esz, cudaMemcpyDeviceToDevice, e->stream));
     }
-    gate_up.w = gu; gate_up.type = type; gate_up.N = 2 * ff; gate_up.K = W;
+    up.w = gu; up.type = type; up.N = per * ff; up.K = W;
     down.w = dn; down.type = type; down.N = W; down.K = ff;
+    return B2_OK;
+}
+
+// two matrices with the same rows side by side: [N][Kl + Kr] (one product forms the sum of both)
+static int side_by_side(b2_engine* e, LayeredModel* m, const std::string& left, int Kl, const std::string& right, int Kr, int N, DenseW& out) {
+    DevTensor tl, tr;
+    int rc;
+    if ((rc = find(e, left, Kl, N, tl)) || (rc = find(e, right, Kr, N, tr))) return rc;
+    if (tl.type != tr.type) return b2_fail(B2_ERR_UNSUPPORTED, left + ", " + right + ": maps whose outputs are added must share a dtype");
+    const size_t esz = tl.type == T_BF16 ? 2 : 4, Kt = (size_t)Kl + Kr;
+    void* cat = nullptr;
+    if ((rc = dev_alloc(m, &cat, (size_t)N * Kt * esz + 64))) return rc;
+    CK(cudaMemcpy2DAsync(cat, Kt * esz, tl.ptr, Kl * esz, Kl * esz, N, cudaMemcpyDeviceToDevice, e->stream));
+    CK(cudaMemcpy2DAsync((char*)cat + Kl * esz, Kt * esz, tr.ptr, Kr * esz, Kr * esz, N, cudaMemcpyDeviceToDevice, e->stream));
+    out.w = cat; out.type = tl.type; out.N = N; out.K = (int)Kt;
     return B2_OK;
 }
 
@@ -277,8 +317,19 @@ int layered_finalize(b2_engine* e) {
     if (c.tie_head) m->head = m->embed;
     else if ((rc = matrix(e, "head", V, W, m->head))) return rc;
     if ((rc = vec_f32(e, m, "final.norm", W, 1, &m->final_norm))) return rc;
-    const bool parallel = c.block_style == B2_BLOCK_PARALLEL_LN;
+    const bool parallel = c.block_style == B2_BLOCK_PARALLEL_LN, one_norm = c.block_style == B2_BLOCK_PARALLEL_ONE_LN;
     if (parallel && (rc = vec_f32(e, m, "final.norm.b", W, 1, &m->final_norm_b))) return rc;
+    if (c.loop_times > 0) {
+        if ((rc = matrix(e, "loop.in", W, 2 * W, m->loop_in))) return rc;
+        if ((rc = vec_f32(e, m, "loop.step", W, c.loop_times, &m->loop_step))) return rc;
+        if ((rc = dev_alloc(m, (void**)&m->loop_x, (size_t)Tm * 2 * W * 4))) return rc;
+    }
+    if (c.embed_sinusoid) {
+        std::vector<double> turns((W + 1) / 2);
+        for (int i = 0; i < (int)turns.size(); i++) turns[i] = pow(10000.0, -2.0 * i / W) / (2.0 * M_PI);
+        if ((rc = dev_alloc(m, (void**)&m->turns, turns.size() * 8))) return rc;
+        CK(cudaMemcpy(m->turns, turns.data(), turns.size() * 8, cudaMemcpyHostToDevice));
+    }
     if (c.bigram_buckets > 0 && (rc = matrix(e, "bigram", c.bigram_buckets + 1, W, m->bigram))) return rc;
     if (c.block_style == B2_BLOCK_PRENORM_RMS && (rc = vec_f32(e, m, "embed.norm", W, 1, &m->embed_norm))) return rc;
     const size_t cache_esz = m->exact ? 4 : 2;
@@ -299,9 +350,12 @@ int layered_finalize(b2_engine* e) {
         if (d.mixer == B2_MIX_SINK_DELTA) {
             if ((rc2 = dev_alloc(m, (void**)&L.st_conv_state, (size_t)S * std::max(1, d.conv_taps - 1) * L.conv_C * 4, true))) return rc2;
             if ((rc2 = dev_alloc(m, (void**)&L.st_state, (size_t)S * col_state_floats(d.mm_heads, d.mm_dim, d.mm_vdim) * 4, true))) return rc2;
+        } else if (d.attn_flags & B2_ATTN_CONV) {
+            if ((rc2 = dev_alloc(m, (void**)&L.st_conv_state, (size_t)S * std::max(1, d.conv_taps - 1) * L.conv_C * 4, true))) return rc2;
         }
         return B2_OK;
     };
+    std::vector<MoeTableLayer> table_layers;
     auto canon_state = [&](LyLayer& L) -> int {
         for (int q = 0; q < 2; q++) {
             L.canon_state[q] = nullptr;
@@ -350,13 +404,20 @@ int layered_finalize(b2_engine* e) {
             const bool two = d.mixer == B2_MIX_SINK_DELTA;
             const std::string a = two ? p + "mix.left." : p + "mix.", b = p + "mix.right.";
             const int H = d.n_head, G = d.n_head_kv, qd = H * d.head_dim, kd = G * d.head_dim, vd = G * d.attn_vdim, od = H * d.attn_vdim;
+            const bool gate = !(d.attn_flags & B2_ATTN_NO_GATE);
             const int gd = (d.attn_flags & B2_ATTN_HEAD_GATE) ? H : od;
             const int Hr = d.mm_heads, rkd = d.key_heads * d.mm_dim, rvd = Hr * d.mm_vdim;
-            std::vector<std::pair<std::string, int>> parts = {{a + "q", qd}, {a + "k", kd}, {a + "v", vd}, {a + "g", gd}};
+            // a gated squared-ReLU shared expert behind the same norm rides along
+            const int sff = one_norm && d.n_ff > 0 && d.ff_kind == B2_FF_MOE && d.moe_expert == B2_EXPERT_RELU2 ? d.moe_shared_ff : 0;
+            std::vector<std::pair<std::string, int>> parts = {{a + "q", qd}, {a + "k", kd}, {a + "v", vd}};
+            if (gate) parts.push_back({a + "g", gd});
             if (two) for (auto& pr : std::vector<std::pair<std::string, int>>{{b + "q", rkd}, {b + "k", rkd}, {b + "v", rvd}, {b + "b", Hr}, {b + "a", Hr}, {b + "g", rvd}}) parts.push_back(pr);
+            if (sff > 0 && d.moe_shared_gate) parts.push_back({p + "mlp.shared.sg", 1});
+            if (sff > 0) parts.push_back({p + "mlp.shared.up", sff});
             std::vector<int> offs;
             if ((rc = fuse(e, m, parts, W, L.sk_proj, offs))) return rc;
-            L.q_off = offs[0]; L.k_off = offs[1]; L.v_off = offs[2]; L.gl_off = offs[3];
+            L.q_off = offs[0]; L.k_off = offs[1]; L.v_off = offs[2]; L.gl_off = gate ? offs[3] : -1;
+            if (sff > 0) { L.su_off = offs.back(); L.sg_off = d.moe_shared_gate ? offs[offs.size() - 2] : -1; }
             if (d.attn_flags & B2_ATTN_BIAS) {       // one bias row for the fused product; the gate has none
                 if ((rc = dev_alloc(m, (void**)&L.sk_bias, (size_t)L.sk_proj.N * 4, true))) return rc;
                 const std::pair<std::string, int> bs[3] = {{a + "q.b", qd}, {a + "k.b", kd}, {a + "v.b", vd}};
@@ -367,9 +428,20 @@ int layered_finalize(b2_engine* e) {
                     CK(cudaGetLastError());
                 }
             }
-            if (e->tensors.count(a + "sink") && (rc = vec_f32(e, m, a + "sink", H, 1, &L.sink))) return rc;
+            if (d.attn_flags & B2_ATTN_UNIT_SINK) { if ((rc = dev_alloc(m, (void**)&L.sink, (size_t)H * 4, true))) return rc; }       // score 0
+            else if (!(d.attn_flags & B2_ATTN_NO_SINK) && e->tensors.count(a + "sink") && (rc = vec_f32(e, m, a + "sink", H, 1, &L.sink))) return rc;
+            if (d.attn_flags & B2_ATTN_FULL_NORM) {
+                if ((rc = vec_f32(e, m, a + "q.norm", qd, 1, &L.q_norm))) return rc;
+                if ((rc = vec_f32(e, m, a + "k.norm", kd, 1, &L.k_norm))) return rc;
+            }
+            if (!two && (d.attn_flags & B2_ATTN_CONV)) {
+                L.conv_off = L.q_off; L.conv_C = qd + kd + vd;
+                if ((rc = concat_f32(e, m, {{a + "q.conv", qd}, {a + "k.conv", kd}, {a + "v.conv", vd}}, d.conv_taps, &L.st_conv_w))) return rc;
+            }
+            if ((d.attn_flags & B2_ATTN_OUT_BIAS) && (rc = vec_f32(e, m, a + "o.b", W, 1, &L.o_bias))) return rc;
             if ((d.attn_flags & B2_ATTN_TALK) && (rc = vec_f32(e, m, a + "talk", H, H, &L.talk))) return rc;
-            if ((rc = matrix(e, a + "o", W, od, L.attn_o))) return rc;
+            if (sff > 0) { if ((rc = side_by_side(e, m, a + "o", od, p + "mlp.shared.down", sff, W, L.attn_o))) return rc; }
+            else if ((rc = matrix(e, a + "o", W, od, L.attn_o))) return rc;
             if ((rc = build_rotary(e, m, L))) return rc;
             if (two) {
                 L.conv_off = offs[4]; L.conv_C = 2 * rkd + rvd; L.b_off = offs[7]; L.ra_off = offs[8]; L.rg_off = offs[9];
@@ -383,7 +455,7 @@ int layered_finalize(b2_engine* e) {
             }
             if ((rc = sink_state(L))) return rc;
             max_proj = std::max<size_t>(max_proj, L.sk_proj.N);
-            max_buf = std::max<size_t>({max_buf, (size_t)qd, (size_t)od, two ? (size_t)L.conv_C : 1, two ? (size_t)rvd : 1});
+            max_buf = std::max<size_t>({max_buf, (size_t)qd, (size_t)od + sff, two ? (size_t)L.conv_C : 1, two ? (size_t)rvd : 1});
             if (d.attn_flags & B2_ATTN_TALK) max_cross = std::max<size_t>(max_cross, (size_t)H * G * d.attn_vdim);
             max_part = std::max<size_t>(max_part, (size_t)H * ((d.attn_flags & B2_ATTN_TALK) ? G : 1) * (d.attn_vdim + 2));
             if ((d.attn_flags & B2_ATTN_TALK) && !m->exact) {       // all tiles of the largest step, up to 512 MB
@@ -475,17 +547,7 @@ int layered_finalize(b2_engine* e) {
             if ((rc = vec_f32(e, m, a + "pb", d.n_head, 1, &L.pb))) return rc;
             if ((rc = vec_f32(e, m, b + "norm", rvd, 1, &L.mm_norm))) return rc;
             if ((rc = vec_f32(e, m, b + "decay", d.mm_heads, 1, &L.decay))) return rc;
-            {   // the two output maps side by side: [W][od + rvd]
-                DevTensor tl, tr;
-                if ((rc = find(e, a + "o", od, W, tl)) || (rc = find(e, b + "o", rvd, W, tr))) return rc;
-                if (tl.type != tr.type) return b2_fail(B2_ERR_UNSUPPORTED, a + "o: the two output maps must share a dtype");
-                const size_t esz = tl.type == T_BF16 ? 2 : 4, Kt = (size_t)od + rvd;
-                void* cat = nullptr;
-                if ((rc = dev_alloc(m, &cat, (size_t)W * Kt * esz + 64))) return rc;
-                CK(cudaMemcpy2DAsync(cat, Kt * esz, tl.ptr, od * esz, od * esz, W, cudaMemcpyDeviceToDevice, e->stream));
-                CK(cudaMemcpy2DAsync((char*)cat + od * esz, Kt * esz, tr.ptr, rvd * esz, rvd * esz, W, cudaMemcpyDeviceToDevice, e->stream));
-                L.cl_o.w = cat; L.cl_o.type = tl.type; L.cl_o.N = W; L.cl_o.K = (int)Kt;
-            }
+            if ((rc = side_by_side(e, m, a + "o", od, b + "o", rvd, W, L.cl_o))) return rc;
             const size_t kpool = (size_t)c.kv_num_blocks * d.n_head_kv * c.kv_block_tokens * d.head_dim * cache_esz;
             const size_t vpool = (size_t)c.kv_num_blocks * d.n_head_kv * c.kv_block_tokens * d.attn_vdim * cache_esz;
             if ((rc = dev_alloc(m, &L.k_pool, kpool, true))) return rc;
@@ -555,24 +617,37 @@ int layered_finalize(b2_engine* e) {
         }
         if (d.n_ff > 0 && d.ff_kind == B2_FF_MOE) {
             const int slots = d.moe_experts + d.moe_identity;
-            if ((rc = vec_f32(e, m, p + "norm2", W, 1, &L.norm2))) return rc;
-            if ((rc = matrix(e, p + "mlp.router", slots, W, L.router))) return rc;
+            if (!one_norm && (rc = vec_f32(e, m, p + "norm2", W, 1, &L.norm2))) return rc;
+            const bool table = d.moe_route == B2_ROUTE_TABLE, relu2 = d.moe_expert == B2_EXPERT_RELU2;
+            if (!table && (rc = matrix(e, p + "mlp.router", slots, W, L.router))) return rc;
             const std::string cn = p + (d.moe_route == B2_ROUTE_TOPK_SOFTMAX ? "mlp.router.b" : "mlp.correction");
-            if ((!(hyper || d.moe_route == B2_ROUTE_SIGMOID) || e->tensors.count(cn)) && (rc = vec_f32(e, m, cn, slots, 1, &L.correction))) return rc;
-            if ((rc = stack_experts(e, m, p + "mlp.e", d.moe_experts, d.n_ff, W, L.gate_up, L.e_down))) return rc;
-            if (d.moe_shared_ff > 0) {
+            if (!table && (!(hyper || d.moe_route == B2_ROUTE_SIGMOID) || e->tensors.count(cn)) && (rc = vec_f32(e, m, cn, slots, 1, &L.correction))) return rc;
+            if ((rc = stack_experts(e, m, p + "mlp.e", d.moe_experts, d.n_ff, W, L.gate_up, L.e_down, !relu2))) return rc;
+            if (table) {
+                MoeTableLayer& pl = L.plan;
+                const size_t pairs = (size_t)Tm * d.moe_top;
+                if ((rc = int_table(e, p + "mlp.table", V, d.moe_top, d.moe_experts, &pl.table))) return rc;
+                pl.top = d.moe_top; pl.n_experts = d.moe_experts; pl.max_tiles = (int)(pairs / 64 + d.moe_experts + 1);
+                pl.big_ok = !m->exact && L.gate_up.type == T_BF16 && W % 8 == 0 && d.n_ff % 8 == 0;
+                int** const bufs[4] = {&pl.sel, &pl.tok, &pl.pos, &pl.x_rows};
+                for (int** b : bufs) if ((rc = dev_alloc(m, (void**)b, pairs * 4, true))) return rc;
+                if ((rc = dev_alloc(m, (void**)&pl.tiles, (size_t)(3 * pl.max_tiles + 1) * 4, true))) return rc;
+                table_layers.push_back(pl);
+                m->table_experts = std::max(m->table_experts, d.moe_experts);
+            }
+            if (d.moe_shared_ff > 0 && !relu2) {
                 if ((rc = stack_experts(e, m, p + "mlp.shared", 0, d.moe_shared_ff, W, L.glu_gate_up, L.glu_down))) return rc;
                 max_glu = std::max<size_t>(max_glu, d.moe_shared_ff);
             }
             moe_pairs = std::max<size_t>(moe_pairs, (size_t)Tm * d.moe_top);
-            moe_slots = std::max<size_t>(moe_slots, slots);
+            if (!table) moe_slots = std::max<size_t>(moe_slots, slots);
             moe_ff = std::max<size_t>(moe_ff, d.n_ff);
             moe_xb = std::max<size_t>(moe_xb, (size_t)d.moe_top * d.n_ff);
             moe_experts = std::max<size_t>(moe_experts, d.moe_experts);
         } else if (d.n_ff > 0 && d.ff_kind == B2_FF_PIECEWISE) {
             float* act = nullptr;
             float host[2] = {0.f, 0.f};
-            if ((rc = vec_f32(e, m, p + "norm2", W, 1, &L.norm2))) return rc;
+            if (!one_norm && (rc = vec_f32(e, m, p + "norm2", W, 1, &L.norm2))) return rc;
             if ((rc = matrix(e, p + "mlp.up", d.n_ff, W, L.up))) return rc;
             if ((rc = matrix(e, p + "mlp.down", W, d.n_ff, L.down))) return rc;
             if ((rc = vec_f32(e, m, p + "mlp.act", 2, 1, &act))) return rc;
@@ -582,17 +657,22 @@ int layered_finalize(b2_engine* e) {
             L.act_p0 = (float)softplus(host[0]); L.act_p1 = (float)(0.5 + softplus(host[1]));
             max_ff = std::max<size_t>(max_ff, d.n_ff);
         } else if (d.n_ff > 0 && d.ff_kind == B2_FF_GLU) {
-            if ((rc = vec_f32(e, m, p + "norm2", W, 1, &L.norm2))) return rc;
+            if (!one_norm && (rc = vec_f32(e, m, p + "norm2", W, 1, &L.norm2))) return rc;
             if ((rc = stack_experts(e, m, p + "mlp", 0, d.n_ff, W, L.glu_gate_up, L.glu_down))) return rc;
             max_glu = std::max<size_t>(max_glu, d.n_ff);
         } else if (d.n_ff > 0) {
-            if ((rc = vec_f32(e, m, p + "norm2", W, 1, &L.norm2))) return rc;
+            if (!one_norm && (rc = vec_f32(e, m, p + "norm2", W, 1, &L.norm2))) return rc;
             if ((rc = matrix(e, p + "mlp.up", d.n_ff, W, L.up))) return rc;
             if ((rc = vec_f32(e, m, p + "mlp.up.b", d.n_ff, 1, &L.up_b))) return rc;
             if ((rc = matrix(e, p + "mlp.down", W, d.n_ff, L.down))) return rc;
             if ((rc = vec_f32(e, m, p + "mlp.down.b", W, 1, &L.down_b))) return rc;
             max_ff = std::max<size_t>(max_ff, d.n_ff);
         }
+    }
+    if (!table_layers.empty()) {
+        m->n_table = (int)table_layers.size();
+        if ((rc = dev_alloc(m, (void**)&m->table_layers, sizeof(MoeTableLayer) * table_layers.size()))) return rc;
+        CK(cudaMemcpy(m->table_layers, table_layers.data(), sizeof(MoeTableLayer) * table_layers.size(), cudaMemcpyHostToDevice));
     }
     if ((rc = dev_alloc(m, (void**)&m->x, (size_t)Tm * W * 4))) return rc;
     if (hyper) {
@@ -612,7 +692,7 @@ int layered_finalize(b2_engine* e) {
     if (parallel && (rc = dev_alloc(m, (void**)&m->hn2, (size_t)Tm * W * 4))) return rc;
     max_ff = std::max(max_ff, max_glu);
     if ((rc = dev_alloc(m, (void**)&m->ff, (size_t)Tm * max_ff * 4))) return rc;
-    if (!m->exact && (rc = dev_alloc(m, (void**)&m->xb, (size_t)(Tm + B2_STEP_MAX_ENTRIES) * std::max<size_t>({max_buf, max_ff, (size_t)W, moe_xb}) * 2 + 64))) return rc;
+    if (!m->exact && (rc = dev_alloc(m, (void**)&m->xb, (size_t)(Tm + B2_STEP_MAX_ENTRIES) * std::max<size_t>({max_buf, max_ff, (size_t)(c.loop_times > 0 ? 2 * W : W), moe_xb}) * 2 + 64))) return rc;
     if (max_part > 0) {                      // sink attention: up to 8 tokens x 16 key ranges
         m->attn_split_floats = (int)std::min<size_t>(max_part * 8 * 16, (size_t)1 << 28);
         if ((rc = dev_alloc(m, (void**)&m->attn_split, (size_t)m->attn_split_floats * 4))) return rc;
@@ -672,8 +752,9 @@ int layered_seq_reset(b2_engine* e, int slot) {
                 const size_t cs = (size_t)std::max(1, m->c.canon_taps - 1) * m->c.n_embd;
                 CK(cudaMemsetAsync(L.canon_state[q] + slot * cs, 0, cs * 4, e->stream));
             }
-        if (d.mixer == B2_MIX_SINK_ATTN) {
-            // nothing but cache pages, which are overwritten
+        if (d.mixer == B2_MIX_SINK_ATTN) {          // cache pages are overwritten
+            const size_t cs = (size_t)std::max(1, d.conv_taps - 1) * L.conv_C;
+            if (L.st_conv_state) CK(cudaMemsetAsync(L.st_conv_state + slot * cs, 0, cs * 4, e->stream));
         } else if (d.mixer == B2_MIX_SINK_DELTA) {
             const size_t cs = (size_t)std::max(1, d.conv_taps - 1) * L.conv_C, ss = col_state_floats(d.mm_heads, d.mm_dim, d.mm_vdim);
             CK(cudaMemsetAsync(L.st_conv_state + slot * cs, 0, cs * 4, e->stream));
@@ -761,7 +842,17 @@ extern "C" int b2_engine_create_layered(const b2_layered_config* c, const b2_lay
                     return b2_fail(B2_ERR_ARG, li + "bad delta-rule sizes");
                 if (d.mm_dim > 256) return b2_fail(B2_ERR_UNSUPPORTED, li + "delta-rule key size above 256");
             }
-            if (c->block_style != B2_BLOCK_HYPER_RMS) return b2_fail(B2_ERR_UNSUPPORTED, li + "this mixer belongs to blocks with stream copies");
+            if (c->block_style != B2_BLOCK_HYPER_RMS && !(d.mixer == B2_MIX_SINK_ATTN && c->block_style == B2_BLOCK_PARALLEL_ONE_LN))
+                return b2_fail(B2_ERR_UNSUPPORTED, li + "this mixer belongs to blocks with stream copies, or (attention alone) to parallel blocks behind one norm");
+            const int own = B2_ATTN_CONV | B2_ATTN_FULL_NORM;
+            if (d.mixer == B2_MIX_SINK_DELTA && (d.attn_flags & own)) return b2_fail(B2_ERR_UNSUPPORTED, li + "convolutions and whole-projection norms belong to the attention alone");
+            if ((d.attn_flags & B2_ATTN_CONV) && (d.conv_taps <= 0 || d.conv_taps > 64)) return b2_fail(B2_ERR_ARG, li + "bad number of taps");
+            const bool side = c->block_style == B2_BLOCK_PARALLEL_ONE_LN && d.moe_shared_ff > 0;
+            if (((d.attn_flags & own) || side) && (d.rot_dims > 0 || (d.attn_flags & B2_ATTN_UNIT_QK)))
+                return b2_fail(B2_ERR_UNSUPPORTED, li + "rotation and unit queries do not go with convolutions, whole-projection norms or a shared expert that rides along");
+            if ((d.attn_flags & B2_ATTN_FULL_NORM) && (int64_t)d.n_head * d.head_dim > 50 * 1024) return b2_fail(B2_ERR_UNSUPPORTED, li + "queries of more than 51200 entries under one norm");
+            if (d.softcap > 0.0 && (d.attn_flags & B2_ATTN_TALK)) return b2_fail(B2_ERR_UNSUPPORTED, li + "capped scores with mixed heads");
+            if (d.qtemp_coef != 0.0 && !(d.qtemp_every > 0.0)) return b2_fail(B2_ERR_ARG, li + "query temperature needs a positive period");
         } else return b2_fail(B2_ERR_UNSUPPORTED, li + "unknown mixer kind");
         if (d.weights_of < 0 || d.weights_of > c->n_layer) return b2_fail(B2_ERR_ARG, li + "weights_of out of range");
         if (d.n_ff > 0 && d.ff_kind == B2_FF_MOE) {
@@ -770,18 +861,26 @@ extern "C" int b2_engine_create_layered(const b2_layered_config* c, const b2_lay
                 d.moe_keep <= 0 || d.moe_keep > d.moe_groups || d.moe_top > d.moe_keep * (slots / d.moe_groups))
                 return b2_fail(B2_ERR_ARG, li + "bad mixture-of-experts sizes");
             if (slots > 4096) return b2_fail(B2_ERR_UNSUPPORTED, li + "more than 4096 expert slots");
-            if (d.moe_route != B2_ROUTE_SOFTMAX_ALL && d.moe_route != B2_ROUTE_TOPK_SOFTMAX && d.moe_route != B2_ROUTE_SIGMOID) return b2_fail(B2_ERR_ARG, li + "unknown routing rule");
+            if (d.moe_route != B2_ROUTE_SOFTMAX_ALL && d.moe_route != B2_ROUTE_TOPK_SOFTMAX && d.moe_route != B2_ROUTE_SIGMOID && d.moe_route != B2_ROUTE_TABLE) return b2_fail(B2_ERR_ARG, li + "unknown routing rule");
+            if (d.moe_route == B2_ROUTE_TABLE && (d.moe_identity > 0 || d.moe_groups > 1 || d.moe_scale_input)) return b2_fail(B2_ERR_UNSUPPORTED, li + "experts by token id have no identity slots, groups or scaled inputs");
+            if (d.moe_expert == B2_EXPERT_RELU2 && d.moe_scale_input) return b2_fail(B2_ERR_UNSUPPORTED, li + "squared-ReLU experts have no scaled input");
+            if (d.moe_shared_ff > 0 && ((d.moe_expert == B2_EXPERT_RELU2) != (d.moe_shared_gate != 0)))
+                return b2_fail(B2_ERR_UNSUPPORTED, li + "a shared expert has a gate if it is a squared-ReLU unit, and none otherwise");
+            if (d.moe_shared_ff > 0 && d.moe_shared_gate && !(c->block_style == B2_BLOCK_PARALLEL_ONE_LN && d.mixer == B2_MIX_SINK_ATTN))
+                return b2_fail(B2_ERR_UNSUPPORTED, li + "a gated shared expert belongs to softmax attention in parallel blocks behind one norm");
             if (d.moe_route == B2_ROUTE_TOPK_SOFTMAX && (d.moe_identity > 0 || d.moe_groups > 1)) return b2_fail(B2_ERR_UNSUPPORTED, li + "top-k softmax routing has no identity slots or groups");
             if (d.moe_scale_input && d.moe_identity > 0) return b2_fail(B2_ERR_UNSUPPORTED, li + "identity slots have no scaled input");
             if (d.moe_shared_ff < 0) return b2_fail(B2_ERR_ARG, li + "negative shared-expert width");
-            if (d.moe_expert != B2_EXPERT_SILU && d.moe_expert != B2_EXPERT_CLAMPED) return b2_fail(B2_ERR_ARG, li + "unknown expert kind");
+            if (d.moe_expert != B2_EXPERT_SILU && d.moe_expert != B2_EXPERT_CLAMPED && d.moe_expert != B2_EXPERT_RELU2) return b2_fail(B2_ERR_ARG, li + "unknown expert kind");
             if (d.moe_expert == B2_EXPERT_CLAMPED && !(d.moe_limit > 0.0)) return b2_fail(B2_ERR_ARG, li + "a clamped expert needs a positive limit");
         } else if (d.ff_kind != B2_FF_RELU2 && d.ff_kind != B2_FF_GLU && d.ff_kind != B2_FF_PIECEWISE) return b2_fail(B2_ERR_UNSUPPORTED, li + "unknown feed-forward kind");
         if (d.ff_act != B2_ACT_SILU && d.ff_act != B2_ACT_GELU_TANH) return b2_fail(B2_ERR_ARG, li + "unknown activation");
-        if ((c->block_style == B2_BLOCK_PRENORM_RMS || c->block_style == B2_BLOCK_PARALLEL_LN) && d.mixer == B2_MIX_WINDOW_SCAN)
+        if (d.loop_pass < 0 || d.loop_pass > c->loop_times || (d.loop_pass > 0 && c->block_style != B2_BLOCK_PARALLEL_ONE_LN && c->block_style != B2_BLOCK_PARALLEL_LN))
+            return b2_fail(B2_ERR_ARG, li + "loop_pass out of range, or not in parallel blocks");
+        if ((c->block_style == B2_BLOCK_PRENORM_RMS || c->block_style == B2_BLOCK_PARALLEL_LN || c->block_style == B2_BLOCK_PARALLEL_ONE_LN) && d.mixer == B2_MIX_WINDOW_SCAN)
             return b2_fail(B2_ERR_UNSUPPORTED, li + "the two-branch mixer belongs to post-sum blocks");
     }
-    if (c->block_style < B2_BLOCK_POSTSUM_LN || c->block_style > B2_BLOCK_PARALLEL_LN)
+    if (c->block_style < B2_BLOCK_POSTSUM_LN || c->block_style > B2_BLOCK_PARALLEL_ONE_LN)
         return b2_fail(B2_ERR_ARG, "unknown block style");
     if (c->block_style == B2_BLOCK_HYPER_RMS) {
         if (c->n_streams < 0 || c->n_streams > 16) return b2_fail(B2_ERR_UNSUPPORTED, "at most 16 copies of the stream");
@@ -792,6 +891,7 @@ extern "C" int b2_engine_create_layered(const b2_layered_config* c, const b2_lay
     }
     if (c->block_style == B2_BLOCK_OUTNORM_RMS && (c->norm_groups < 0 || (c->norm_groups > 0 && c->n_embd % c->norm_groups)))
         return b2_fail(B2_ERR_ARG, "the norm's parts must divide the width");
+    if (c->loop_times < 0) return b2_fail(B2_ERR_ARG, "negative number of passes");
     if (c->bigram_buckets < 0 || c->bigram_mul_prev < 0 || c->bigram_mul_cur < 0) return b2_fail(B2_ERR_ARG, "bad bigram embedding");
     b2_engine* e = new b2_engine();
     b2_config& b = e->cfg;
@@ -1096,16 +1196,22 @@ static int mix_sink(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& 
     const b2_layered_config& c = m->c;
     const b2_layer_desc& d = L.d;
     cudaStream_t st = e->stream;
-    const int T = r.T, W = c.n_embd, Np = L.sk_proj.N, H = d.n_head, od = H * d.attn_vdim;
+    const int T = r.T, W = c.n_embd, Np = L.sk_proj.N, H = d.n_head, od = H * d.attn_vdim, Ko = L.attn_o.K;
     int rc;
-    if ((rc = dense(e, m, L.sk_proj, in, W, m->proj, Np, T, L.sk_bias, L.sk_bias ? EPI_BIAS : EPI_NONE))) return rc;
+    DenseArgs pj = {};
+    pj.n_act = L.su_off;                   // the rows of a shared expert that rides along get their activation here
+    if ((rc = dense(e, m, L.sk_proj, in, W, m->proj, Np, T, L.sk_bias, L.su_off >= 0 ? EPI_BIAS_TAIL_RELU2 : L.sk_bias ? EPI_BIAS : EPI_NONE, 1, &pj))) return rc;
     SinkAttnArgs a = {};
     a.proj = m->proj; a.ldp = Np; a.q_off = L.q_off; a.k_off = L.k_off; a.v_off = L.v_off;
     a.rot.cos = L.rot_cos; a.rot.sin = L.rot_sin; a.rot.rot_dims = d.rot_dims; a.unit_qk = (d.attn_flags & B2_ATTN_UNIT_QK) ? 1 : 0;
     a.k_pool = L.k_pool; a.v_pool = L.v_pool; a.cache_f32 = m->exact ? 1 : 0; a.block_tables = m->block_tables; a.block_tokens = c.kv_block_tokens;
     a.H = H; a.G = d.n_head_kv; a.d = d.head_dim; a.dv = d.attn_vdim; a.window = d.window; a.scale = (float)d.attn_scale; a.eps = c.norm_eps;
-    a.sink = L.sink; a.talk = L.talk; a.gate = m->proj + L.gl_off; a.ld_gate = Np; a.gate_per_head = (d.attn_flags & B2_ATTN_HEAD_GATE) ? 1 : 0;
-    a.q_rot = m->buf[0]; a.cross = m->cross; a.out = m->buf[1]; a.ld_out = od;
+    a.sink = L.sink; a.talk = L.talk; a.gate = L.gl_off >= 0 ? m->proj + L.gl_off : nullptr; a.ld_gate = Np; a.gate_per_head = (d.attn_flags & B2_ATTN_HEAD_GATE) ? 1 : 0;
+    a.q_rot = m->buf[0]; a.cross = m->cross; a.out = m->buf[1]; a.ld_out = Ko;
+    a.softcap = (float)d.softcap; a.temp_coef = (float)d.qtemp_coef; a.temp_every = d.qtemp_every;
+    a.q_norm_w = L.q_norm; a.k_norm_w = L.k_norm;
+    if (d.attn_flags & B2_ATTN_CONV) { a.conv_w = L.st_conv_w; a.taps = d.conv_taps; a.conv_state = L.st_conv_state; }
+    if (L.su_off >= 0) { a.side_off = L.su_off; a.side_gate = L.sg_off; a.side_n = Ko - od; a.side_col = od; }
     a.pbuf = m->attn_pbuf; a.pbuf_floats = m->attn_pbuf_floats;
     a.part = m->attn_split; a.part_capacity = m->attn_split_floats; a.max_keys = d.window > 0 ? std::min(d.window, c.n_ctx) : c.n_ctx;
     {
@@ -1114,7 +1220,7 @@ static int mix_sink(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& 
         CK(sink_attn_launch(a, r, st));
         e->launches += L.talk ? 3 : 2;
     }
-    if ((rc = dense(e, m, L.attn_o, m->buf[1], od, m->oL, W, T))) return rc;
+    if ((rc = dense(e, m, L.attn_o, m->buf[1], Ko, m->oL, W, T, L.o_bias, L.o_bias ? EPI_BIAS : EPI_NONE))) return rc;
     if (d.mixer != B2_MIX_SINK_DELTA) return B2_OK;
     const int Hr = d.mm_heads, G = d.key_heads, kd = G * d.mm_dim, vd = Hr * d.mm_vdim;
     ConvArgs cv = {};
@@ -1180,56 +1286,65 @@ static int ff_moe(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r,
     cudaStream_t st = e->stream;
     const int T = r.T, W = m->c.n_embd, slots = d.moe_experts + d.moe_identity, pairs = T * d.moe_top, ff = d.n_ff;
     int rc;
-    DenseArgs ex = {};
-    ex.exact = true;                               // router scores are 32-bit products in both modes
-    if ((rc = dense(e, m, L.router, in, W, m->moe_logits, slots, T, nullptr, EPI_NONE, 7, &ex))) return rc;
-    MoeRouteArgs ra = {};
-    ra.logits = m->moe_logits; ra.ld = slots; ra.correction = L.correction; ra.n_slots = slots; ra.n_experts = d.moe_experts;
-    ra.top = d.moe_top; ra.n_groups = d.moe_groups; ra.keep_groups = d.moe_keep; ra.scale = (float)d.moe_scale;
-    ra.mode = d.moe_route == B2_ROUTE_TOPK_SOFTMAX ? 1 : d.moe_route == B2_ROUTE_SIGMOID ? 2 : 0; ra.renorm = d.moe_renorm;
-    ra.sel = m->moe_sel; ra.weight = m->moe_weight; ra.pair_token = m->moe_tok;
     DenseGroups g = {};
     g.n_groups = d.moe_experts;
-    const bool tiled = T > 8;
+    const bool tiled = T > MOE_FEW_TOKENS, table = d.moe_route == B2_ROUTE_TABLE;
     // long prompts in the serving mode: 128-row tiles through the large tensor-core kernel
-    const bool big = tiled && !m->exact && L.gate_up.type == T_BF16 && pairs >= 1024 && W % 8 == 0 && ff % 8 == 0 && m->xb;
+    const bool big = tiled && !m->exact && L.gate_up.type == T_BF16 && pairs >= MOE_BIG_PAIRS && W % 8 == 0 && ff % 8 == 0 && m->xb;
     g.tile_max = big ? 128 : 64;
-    {
+    const int *sel = m->moe_sel, *tok = m->moe_tok, *pos = m->moe_pos, *x_rows = m->moe_rows, *tiles = m->moe_tiles;
+    int max_tiles = m->moe_max_tiles;
+    if (table) {                                   // chosen and sorted at the start of the step
+        sel = L.plan.sel; tok = L.plan.tok; pos = L.plan.pos; x_rows = L.plan.x_rows; tiles = L.plan.tiles; max_tiles = L.plan.max_tiles;
+    } else {
+        DenseArgs ex = {};
+        ex.exact = true;                           // router scores are 32-bit products in both modes
+        if ((rc = dense(e, m, L.router, in, W, m->moe_logits, slots, T, nullptr, EPI_NONE, 7, &ex))) return rc;
+        MoeRouteArgs ra = {};
+        ra.logits = m->moe_logits; ra.ld = slots; ra.correction = L.correction; ra.n_slots = slots; ra.n_experts = d.moe_experts;
+        ra.top = d.moe_top; ra.n_groups = d.moe_groups; ra.keep_groups = d.moe_keep; ra.scale = (float)d.moe_scale;
+        ra.mode = d.moe_route == B2_ROUTE_TOPK_SOFTMAX ? 1 : d.moe_route == B2_ROUTE_SIGMOID ? 2 : 0; ra.renorm = d.moe_renorm;
+        ra.sel = m->moe_sel; ra.weight = m->moe_weight; ra.pair_token = m->moe_tok;
         StepProfiler sp(m, st, 7);
         CK(moe_route_launch(ra, T, st));
         e->launches++;
         if (tiled) {
             MoeSortArgs sa = {};
             sa.sel = m->moe_sel; sa.n_pairs = pairs; sa.top = d.moe_top; sa.n_experts = d.moe_experts; sa.tile = g.tile_max; sa.pos = m->moe_pos; sa.x_rows = m->moe_rows;
-            sa.n_tiles = m->moe_tiles; sa.tile_group = m->moe_tiles + 1; sa.tile_row0 = sa.tile_group + m->moe_max_tiles;
-            sa.tile_rows = sa.tile_row0 + m->moe_max_tiles; sa.max_tiles = m->moe_max_tiles;
+            sa.n_tiles = m->moe_tiles; sa.tile_group = m->moe_tiles + 1; sa.tile_row0 = sa.tile_group + max_tiles;
+            sa.tile_rows = sa.tile_row0 + max_tiles; sa.max_tiles = max_tiles;
             if (d.moe_scale_input) { sa.weight = m->moe_weight; sa.row_weight = m->moe_row_weight; }
             CK(moe_sort_launch(sa, st));
             e->launches++;
-            g.tile_group = sa.tile_group; g.tile_row0 = sa.tile_row0; g.tile_rows = sa.tile_rows; g.n_tiles = sa.n_tiles;
-            g.max_tiles = std::min(m->moe_max_tiles, pairs / g.tile_max + d.moe_experts + 1);
-        } else g.group = m->moe_sel;
+        }
     }
+    if (tiled) {
+        g.n_tiles = tiles; g.tile_group = tiles + 1; g.tile_row0 = g.tile_group + max_tiles; g.tile_rows = g.tile_row0 + max_tiles;
+        g.max_tiles = std::min(max_tiles, pairs / g.tile_max + d.moe_experts + 1);
+    } else g.group = sel;
     // weights on the inputs: w (W h) for W (w h), inside the epilogue before the activation; the outputs then add up as they are
-    const float* out_weight = d.moe_scale_input ? nullptr : m->moe_weight;
+    // (experts by token id share one weight, which the down product's epilogue applies)
+    const float* out_weight = d.moe_scale_input || table ? nullptr : m->moe_weight;
     if (d.moe_scale_input) g.row_scale = tiled ? m->moe_row_weight : m->moe_weight;
     DenseArgs up = {};
-    g.x_rows = tiled ? m->moe_rows : m->moe_tok; g.w_stride = (long)2 * ff * W; g.x_total_rows = T;
+    g.x_rows = tiled ? x_rows : tok; g.w_stride = (long)L.gate_up.N * W; g.x_total_rows = T;
     up.groups = &g;
     up.p0 = (float)d.moe_limit; up.p1 = (float)d.moe_alpha;
-    if ((rc = dense(e, m, L.gate_up, in, W, m->moe_h, ff, pairs, nullptr, d.moe_expert == B2_EXPERT_CLAMPED ? EPI_GLU_CLAMP : EPI_GLU_SILU, 1, &up))) return rc;
+    const int act = d.moe_expert == B2_EXPERT_CLAMPED ? EPI_GLU_CLAMP : d.moe_expert == B2_EXPERT_RELU2 ? EPI_BIAS_RELU2 : EPI_GLU_SILU;
+    if ((rc = dense(e, m, L.gate_up, in, W, m->moe_h, ff, pairs, nullptr, act, 1, &up))) return rc;
     DenseGroups g2 = g;
     g2.x_rows = nullptr; g2.row_scale = nullptr; g2.w_stride = (long)W * ff; g2.x_total_rows = pairs;
     DenseArgs dn = {};
     dn.groups = &g2;
+    if (table) dn.scale = 1.f / (float)d.moe_top;
     if ((rc = dense(e, m, L.e_down, m->moe_h, ff, m->moe_y, W, pairs, nullptr, EPI_NONE, 1, &dn))) return rc;
     if (defer) {
-        defer->sel = m->moe_sel; defer->weight = out_weight; defer->pos = tiled ? m->moe_pos : nullptr; defer->rows = m->moe_y; defer->h = in;
+        defer->sel = sel; defer->weight = out_weight; defer->pos = tiled ? pos : nullptr; defer->rows = m->moe_y; defer->h = in;
         defer->n_experts = d.moe_experts; defer->top = d.moe_top;
         return B2_OK;
     }
     StepProfiler sp(m, st, 7);
-    CK(moe_combine_launch(m->moe_sel, out_weight, tiled ? m->moe_pos : nullptr, m->moe_y, in, d.moe_experts, d.moe_top, W, T, out, st));
+    CK(moe_combine_launch(sel, out_weight, tiled ? pos : nullptr, m->moe_y, in, d.moe_experts, d.moe_top, W, T, out, st));
     e->launches++;
     return B2_OK;
 }
@@ -1262,12 +1377,23 @@ static int run_layers(b2_engine* e, LayeredModel* m, const RaggedDev& r) {
         StepProfiler sp(m, st, 0);
         BigramTable bg;
         bg.table = m->bigram.w; bg.w_type = m->bigram.type; bg.buckets = c.bigram_buckets; bg.mul_prev = c.bigram_mul_prev; bg.mul_cur = c.bigram_mul_cur;
-        CK(embed_ragged_launch(m->embed.w, m->embed.type, W, r.tok_id, T, m->x, c.embed_scale != 0.f ? c.embed_scale : 1.f, st, r.tok_prev, &bg));
+        EmbedExtra ex;
+        ex.turns = m->turns; ex.tok_pos = r.tok_pos;
+        if (m->loop_x) {                   // the embedding output stays beside the stream for the passes' input maps
+            ex.ld_copy = 2 * W; ex.copy[0] = m->loop_x + W;
+            if (m->layers[0].d.loop_pass > 0) ex.copy[1] = m->loop_x;
+        }
+        CK(embed_ragged_launch(m->embed.w, m->embed.type, W, r.tok_id, T, m->x, c.embed_scale != 0.f ? c.embed_scale : 1.f, st, r.tok_prev, &bg, &ex));
         e->launches++;
         if (prenorm) {
             CK(resid_rms_norm_launch(m->x, nullptr, 0.f, m->embed_norm, 1.f, 1.f, c.norm_eps, W, T, m->x, st));
             e->launches++;
         }
+    }
+    if (m->n_table > 0) {
+        StepProfiler sp(m, st, 7);
+        CK(moe_table_launch(m->table_layers, m->n_table, m->table_experts, r.tok_id, T, st));
+        e->launches++;
     }
     // pre-norm blocks: a branch output waits in m->oL until the next norm (or the end of the layer) adds it to the stream
     // (a mixture's weighted sum is not even formed before: the same kernel adds it up)
@@ -1335,36 +1461,56 @@ static int run_layers(b2_engine* e, LayeredModel* m, const RaggedDev& r) {
         }
         return B2_OK;
     }
-    if (c.block_style == B2_BLOCK_PARALLEL_LN) {
-        // One kernel per boundary: both outputs of a layer join the stream, and the two norms of the next layer are made from it
-        // (m->hn for the mixer, m->hn2 for the feed-forward block).
+    if (c.block_style == B2_BLOCK_PARALLEL_LN || c.block_style == B2_BLOCK_PARALLEL_ONE_LN) {
+        // One kernel per boundary: both outputs of a layer join the stream, and the norm or norms of the next layer are made from it
+        // (m->hn for the mixer, m->hn2 for the feed-forward block when it has a norm of its own). Where a pass over a run of layers
+        // starts, the sum goes beside the embedding output instead, one product maps the pair to the new stream (the pass's vector
+        // is its bias), and the norm follows.
+        const bool one_norm = c.block_style == B2_BLOCK_PARALLEL_ONE_LN;
+        float* ff_in = one_norm ? m->hn : m->hn2;
         ParallelJoinArgs pj = {};
         MoeJoinArgs pj_moe = {};
+        auto boundary = [&]() -> int {
+            StepProfiler sp(m, st, 5);
+            pj.x = m->x; pj.eps = c.norm_eps; pj.moe = pj_moe.sel ? &pj_moe : nullptr;
+            CK(parallel_join_launch(pj, W, T, st));
+            e->launches++;
+            pj = ParallelJoinArgs{}; pj_moe = MoeJoinArgs{};
+            return B2_OK;
+        };
         for (int li = 0; li <= c.n_layer; li++) {
-            {
-                StepProfiler sp(m, st, 5);
-                pj.x = m->x; pj.eps = c.norm_eps; pj.moe = pj_moe.sel ? &pj_moe : nullptr;
-                if (li < c.n_layer) {
-                    const LyLayer& L = m->layers[li];
-                    pj.w1 = L.norm1; pj.b1 = L.norm1_b; pj.y1 = m->hn;
-                    if (L.d.n_ff > 0) { pj.w2 = L.norm2; pj.b2 = L.norm2_b; pj.y2 = m->hn2; }
+            const LyLayer* next = li < c.n_layer ? &m->layers[li] : nullptr;
+            const bool pass = next && next->d.loop_pass > 0;
+            if (pass) {
+                if (li > 0) {                       // ahead of the first layer the embedding has written both halves
+                    pj.x_copy = m->loop_x; pj.ld_copy = 2 * W;
+                    if ((rc = boundary())) return rc;
                 }
-                CK(parallel_join_launch(pj, W, T, st));
-                e->launches++;
-                pj = ParallelJoinArgs{}; pj_moe = MoeJoinArgs{};
+            } else {
+                if (next) {
+                    pj.w1 = next->norm1; pj.b1 = next->norm1_b; pj.y1 = m->hn;
+                    if (!one_norm && next->d.n_ff > 0) { pj.w2 = next->norm2; pj.b2 = next->norm2_b; pj.y2 = m->hn2; }
+                }
+                if ((rc = boundary())) return rc;
             }
             if (m->trace && li > 0)
                 CK(cudaMemcpyAsync(m->trace + ((size_t)(li - 1) * c.max_step_tokens) * W, m->x, (size_t)T * W * 4, cudaMemcpyDeviceToDevice, st));
-            if (li == c.n_layer) break;
+            if (!next) break;
+            if (pass) {
+                if ((rc = dense(e, m, m->loop_in, m->loop_x, 2 * W, m->x, W, T, m->loop_step + (size_t)(next->d.loop_pass - 1) * W, EPI_BIAS))) return rc;
+                pj.w1 = next->norm1; pj.b1 = next->norm1_b; pj.y1 = m->hn;
+                if (!one_norm && next->d.n_ff > 0) { pj.w2 = next->norm2; pj.b2 = next->norm2_b; pj.y2 = m->hn2; }
+                if ((rc = boundary())) return rc;
+            }
             LyLayer& L = m->layers[li];
             if ((rc = run_mixer(e, m, L, r, m->hn))) return rc;
             pj.a = m->oL;
             if (L.d.n_ff > 0) {
                 const bool moe = L.d.ff_kind == B2_FF_MOE;
-                if ((rc = run_ff(e, m, L, r, m->hn2, m->oR, moe ? &pj_moe : nullptr))) return rc;
+                if ((rc = run_ff(e, m, L, r, ff_in, m->oR, moe ? &pj_moe : nullptr))) return rc;
                 if (!moe) pj.b = m->oR;
-                else if (L.d.moe_shared_ff > 0) {
-                    if ((rc = ff_glu(e, m, L, r, m->hn2, m->oR))) return rc;
+                else if (L.d.moe_shared_ff > 0 && L.su_off < 0) {        // a shared expert that does not ride along with the mixer
+                    if ((rc = ff_glu(e, m, L, r, ff_in, m->oR))) return rc;
                     pj.b = m->oR;
                 }
             }

@@ -35,8 +35,9 @@ struct RaggedDev {             // device pointers, valid for one step
 // EPI_GLU_GELU: the same with the tanh form of GELU.
 // EPI_MUL_SIGMOID: the product times sigmoid(aux[t][n]) (aux_one: sigmoid(aux[t][0]) for all columns of a batch entry).
 // EPI_GLU_CLAMP: pairs as above; g = min(gate, p0), u = clamp(up, -p0, p0); output = g * sigmoid(p1 * g) * (u + 1).
+// EPI_BIAS_TAIL_RELU2: bias (if any), then columns n >= n_act through the squared ReLU (a fused matrix whose last rows feed one).
 // EPI_PIECEWISE: z > 0: p0 z^2 + z / 2; else p1 (exp(z) - 1 - z) + z / 2.
-enum DenseEpi { EPI_NONE = 0, EPI_BIAS = 1, EPI_BIAS_RELU2 = 2, EPI_GLU_SILU = 3, EPI_MUL_SIGMOID = 4, EPI_GLU_CLAMP = 5, EPI_PIECEWISE = 6, EPI_GLU_GELU = 7 };
+enum DenseEpi { EPI_NONE = 0, EPI_BIAS = 1, EPI_BIAS_RELU2 = 2, EPI_GLU_SILU = 3, EPI_MUL_SIGMOID = 4, EPI_GLU_CLAMP = 5, EPI_PIECEWISE = 6, EPI_GLU_GELU = 7, EPI_BIAS_TAIL_RELU2 = 8 };
 // Grouped products (mixture of experts): the rows of a step's (token, choice) pairs, each against the matrix of its group.
 //   tiles == nullptr: row p of the product is pair p itself, blockIdx.y walks the pairs one by one (few-token steps);
 //   else: pairs sorted by group, tile i = rows [tile_row0[i], + tile_rows[i]) of group tile_group[i]; *n_tiles of them.
@@ -65,6 +66,7 @@ struct DenseArgs {
     bool exact;                     // true: 32-bit multiply-adds (no tensor cores, inputs not rounded)
     __nv_bfloat16* xb;              // scratch [T][K] for X rounded to bf16 (large tensor-core steps); null: not available
     float scale = 1.f;              // the product (after the epilogue) times this
+    int n_act = 0;                  // EPI_BIAS_TAIL_RELU2
     float p0 = 0.f, p1 = 0.f;       // constants of EPI_GLU_CLAMP / EPI_PIECEWISE
     const float* aux = nullptr; int ldaux = 0; bool aux_one = false;      // EPI_MUL_SIGMOID
     // batch > 1: `batch` independent products, operand b at x + b * x_bs, w + b * w_bs (elements), y + b * y_bs, aux + b * aux_bs
@@ -75,13 +77,19 @@ struct DenseArgs {
 cudaError_t dense_launch(const DenseArgs& a, cudaStream_t s);
 
 // ---------------------------------------------------------------- mixers and norms (mixers.cu)
-// x[t] = table[tok_id[t]] * scale (+ bigram row of (tok_prev[t], tok_id[t]))
+// x[t] = table[tok_id[t]] * scale (+ bigram row of (tok_prev[t], tok_id[t])) (+ a sinusoid of the position)
 struct BigramTable {           // row (prev * mul_prev + cur * mul_cur) mod buckets; row `buckets` for a sequence's first token
     const void* table = nullptr; int w_type = 0;
     int buckets = 0, mul_prev = 0, mul_cur = 0;
 };
+struct EmbedExtra {
+    const double* turns = nullptr;     // sinusoid: turns per position of pair i, [(W + 1) / 2] (entry 2i: sin, 2i + 1: cos); null: none
+    const int* tok_pos = nullptr;
+    float* copy[2] = {};               // the result also goes here (row stride ld_copy); null: not
+    int ld_copy = 0;
+};
 cudaError_t embed_ragged_launch(const void* table, int w_type, int W, const int* tok_id, int T, float* x, float scale, cudaStream_t s,
-                                const int* tok_prev = nullptr, const BigramTable* bigram = nullptr);
+                                const int* tok_prev = nullptr, const BigramTable* bigram = nullptr, const EmbedExtra* extra = nullptr);
 // gather rows: y[i] = x[rows[i]]
 cudaError_t gather_rows_launch(const float* x, int W, const int* rows, int n, float* y, cudaStream_t s);
 
@@ -255,12 +263,23 @@ struct MoeRouteArgs {
 cudaError_t moe_route_launch(const MoeRouteArgs& a, int T, cudaStream_t s);
 // pairs sorted by expert into tiles of `tile` rows: pos[p] = row of pair p in the sorted order (-1: identity slot), x_rows[row] =
 // token of that row, and the tile table; all in device memory (meta: [0] = number of tiles)
+// (also: a table of token ids instead of a choice, MoeTableLayer)
 struct MoeSortArgs {
     const int* sel; int n_pairs, top, n_experts, tile;      // tile: rows per tile
     int* pos; int* x_rows; int* tile_group; int* tile_row0; int* tile_rows; int* n_tiles; int max_tiles;
     const float* weight = nullptr; float* row_weight = nullptr;      // weight != null: row_weight[row of pair p] = weight[p]
 };
 cudaError_t moe_sort_launch(const MoeSortArgs& a, cudaStream_t s);
+// Experts by token id: the choice of every layer is known before the first layer runs, so ONE launch at the start of a step (a CTA
+// per layer) writes all layers' choices, and for steps with more than MOE_FEW_TOKENS tokens their sorted pair tables too.
+struct MoeTableLayer {
+    const int* table; int top, n_experts;   // [n_vocab][top]
+    int big_ok;                             // 128-row tiles when the step has at least MOE_BIG_PAIRS pairs
+    int *sel, *tok, *pos, *x_rows, *tiles;  // tiles: [0] number of tiles, then group, first row, rows (max_tiles each)
+    int max_tiles;
+};
+constexpr int MOE_FEW_TOKENS = 8, MOE_BIG_PAIRS = 1024;
+cudaError_t moe_table_launch(const MoeTableLayer* dev_layers, int n_layers, int max_experts, const int* tok_id, int T, cudaStream_t s);
 // out[t] = sum over the token's choices, in choice order, of weight * (expert output row | h[t] for identity slots)
 cudaError_t moe_combine_launch(const int* sel, const float* weight, const int* pos, const float* rows, const float* h, int n_experts,
                                int top, int W, int T, float* out, cudaStream_t s);
@@ -275,12 +294,14 @@ cudaError_t moe_join_launch(const MoeJoinArgs& j, float* x, float mult, const fl
                             cudaStream_t s);
 
 // Parallel blocks: x[t] += a[t] + (b[t], or a mixture's sum of expert rows); then every norm given, all of the new x[t]:
-// y = (x - mean) / sqrt(var + eps) * w + bias. Any part may be absent (a == b == moe == null: x stays as it is).
+// y = (x - mean) / sqrt(var + eps) * w + bias (bias may be null). Any part may be absent (a == b == moe == null: x stays as it is).
+// x_copy: the new stream also goes there (row stride ld_copy).
 struct ParallelJoinArgs {
     float* x; const float* a; const float* b; const MoeJoinArgs* moe;
     const float *w1, *b1; float* y1;
     const float *w2, *b2; float* y2;
     float eps;
+    float* x_copy; int ld_copy;
 };
 cudaError_t parallel_join_launch(const ParallelJoinArgs& a, int W, int T, cudaStream_t s);
 
@@ -318,11 +339,21 @@ cudaError_t sigmoid_attn_launch(const SigmoidAttnArgs& a, const RaggedDev& r, cu
 // and k after the rotation, and one extra term exp(sink[h]) in every head's denominator (no key, no value). With `talk` the
 // normalised weights of the heads are mixed, weight_h <- sum_g talk[h][g] weight_g, before head h applies them to the values
 // of ITS key/value head: the kernels then compute A[g][c] = sum_j weight_g(j) v_c(j) for every (query head g, value head c)
-// and a small pass forms out_h = gate_h * sum_g talk[h][g] A[g][c(h)]. The value size may differ from the key size.
+// and a small pass forms out_h = gate_h * sum_g talk[h][g] A[g][c(h)]. The value size may differ from the key size. softcap > 0:
+// scores s <- softcap * tanh(s / softcap) before the softmax (not together with talk).
+// Input preparation beyond rotation and unit RMS (sink_attn_prepare; without those two): a causal convolution over the last `taps`
+// tokens on every channel of q | k | v (neighbouring columns from q_off), RMS norm of q and of k over ALL their heads, and `side`
+// columns: out[t][side_col + i] = proj[t][side_off + i] * sigmoid(proj[t][side_gate]), which puts a gated hidden row of another
+// branch beside the heads' outputs so that one product maps both.
 struct SinkAttnArgs {
     const float* proj; int ldp; int q_off, k_off, v_off;      // projection rows: q [H*d], k [G*d], v [G*dv]
     RotaryTable rot;                                           // pairs (i, i + rot_dims / 2)
     int unit_qk;
+    float softcap;                                             // <= 0: none
+    float temp_coef; double temp_every;                        // q at position p times 1 + coef * ln(floor((p + 1) / every) + 1); coef 0: off
+    const float* q_norm_w; const float* k_norm_w;              // [H*d], [G*d]: whole-projection norms, or null
+    const float* conv_w; int taps; float* conv_state;          // [C][taps], state [slot][taps-1][C], C = H*d + G*d + G*dv; null: none
+    int side_off, side_gate, side_n, side_col;                 // side_n == 0: none
     void* k_pool; void* v_pool; int cache_f32;                 // pages [page][G][block_tokens][d] and [page][G][block_tokens][dv]
     int* const* block_tables; int block_tokens;
     int H, G, d, dv, window;
@@ -337,7 +368,8 @@ struct SinkAttnArgs {
     float* pbuf; size_t pbuf_floats;                           // prompts with mixed heads: the normalised weights of a group of query tiles
     float* out; int ld_out;                                    // out[t][h*dv + i]
 };
-// rotation (and unit RMS) of q and k, keys and values into the pages
+// rotation (and unit RMS) of q and k, or the preparation above; keys and values into the pages; the convolution's state moves on
+bool sink_attn_prepares(const SinkAttnArgs& a);       // sink_attn_store_launch takes the preparation path
 cudaError_t sink_attn_store_launch(const SinkAttnArgs& a, const RaggedDev& r, cudaStream_t s);
 cudaError_t sink_attn_launch(const SinkAttnArgs& a, const RaggedDev& r, cudaStream_t s);
 

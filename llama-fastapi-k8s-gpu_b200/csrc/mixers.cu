@@ -44,7 +44,7 @@ __device__ __forceinline__ float log_sigmoid_f(float z) { return -softplus_f(-z)
 // ---------------------------------------------------------------- embedding, gather
 template <typename TW>
 __global__ void embed_ragged_kernel(const TW* __restrict__ table, int W, const int* __restrict__ tok, float* __restrict__ x, float scale,
-                                    const int* __restrict__ tok_prev, BigramTable bg) {
+                                    const int* __restrict__ tok_prev, BigramTable bg, EmbedExtra ex) {
     griddep_launch();
     griddep_wait();
     const int t = blockIdx.x, cur = tok[t];
@@ -62,15 +62,22 @@ __global__ void embed_ragged_kernel(const TW* __restrict__ table, int W, const i
             const size_t j = pair_row * W + i;
             v += bg.w_type == T_BF16 ? __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(bg.table)[j]) : reinterpret_cast<const float*>(bg.table)[j];
         }
+        if (ex.turns) {                       // whole turns are dropped in double precision, so far positions lose nothing
+            const double a = (double)ex.tok_pos[t] * ex.turns[i >> 1];
+            const float half_turns = (float)(2.0 * (a - rint(a)));
+            v += i & 1 ? cospif(half_turns) : sinpif(half_turns);
+        }
         x[(size_t)t * W + i] = v;
+        for (int k = 0; k < 2; k++) if (ex.copy[k]) ex.copy[k][(size_t)t * ex.ld_copy + i] = v;
     }
 }
 cudaError_t embed_ragged_launch(const void* table, int w_type, int W, const int* tok_id, int T, float* x, float scale, cudaStream_t s,
-                                const int* tok_prev, const BigramTable* bigram) {
+                                const int* tok_prev, const BigramTable* bigram, const EmbedExtra* extra) {
+    const EmbedExtra ex = extra ? *extra : EmbedExtra{};
     const BigramTable bg = bigram ? *bigram : BigramTable{};
     if (bg.table && !tok_prev) return cudaErrorInvalidValue;
-    if (w_type == T_BF16) return launch_chain(embed_ragged_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, s, (const __nv_bfloat16*)table, W, tok_id, x, scale, tok_prev, bg);
-    if (w_type == T_F32) return launch_chain(embed_ragged_kernel<float>, dim3(T), dim3(128), 0, s, (const float*)table, W, tok_id, x, scale, tok_prev, bg);
+    if (w_type == T_BF16) return launch_chain(embed_ragged_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, s, (const __nv_bfloat16*)table, W, tok_id, x, scale, tok_prev, bg, ex);
+    if (w_type == T_F32) return launch_chain(embed_ragged_kernel<float>, dim3(T), dim3(128), 0, s, (const float*)table, W, tok_id, x, scale, tok_prev, bg, ex);
     return cudaErrorInvalidValue;
 }
 
@@ -190,6 +197,7 @@ __global__ void __launch_bounds__(NT) parallel_join_kernel(ParallelJoinDev p, in
             y += acc;
         }
         if (adds) { v += y; a.x[base + i] = v; }
+        if (a.x_copy) a.x_copy[(size_t)t * a.ld_copy + i] = v;
         row[i] = v;
         sum += v;
     }
@@ -200,8 +208,8 @@ __global__ void __launch_bounds__(NT) parallel_join_kernel(ParallelJoinDev p, in
     const float rstd = 1.f / sqrtf(block_sum(sq, red) / (float)W + a.eps);
     for (int i = threadIdx.x; i < W; i += NT) {
         const float u = (row[i] - mean) * rstd;
-        if (a.y1) a.y1[base + i] = fmaf(u, a.w1[i], a.b1[i]);
-        if (a.y2) a.y2[base + i] = fmaf(u, a.w2[i], a.b2[i]);
+        if (a.y1) a.y1[base + i] = fmaf(u, a.w1[i], a.b1 ? a.b1[i] : 0.f);
+        if (a.y2) a.y2[base + i] = fmaf(u, a.w2[i], a.b2 ? a.b2[i] : 0.f);
     }
 }
 cudaError_t parallel_join_launch(const ParallelJoinArgs& a, int W, int T, cudaStream_t s) {

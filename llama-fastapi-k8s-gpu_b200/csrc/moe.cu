@@ -1,5 +1,5 @@
 // Mixture of experts for the layer-list models: routing (softmax or sigmoid scores, additive choice correction, group-limited
-// top-k with identity slots; or biased logits with a softmax over the chosen ones), the bookkeeping that sorts a step's (token, choice) pairs by expert into row tiles for the
+// top-k with identity slots; or biased logits with a softmax over the chosen ones; or a table of token ids), the bookkeeping that sorts a step's (token, choice) pairs by expert into row tiles for the
 // grouped products of dense.cu, and the weighted combination. Routing arithmetic is 32-bit.
 #include "kernels.h"
 #include "layered.h"
@@ -128,11 +128,8 @@ cudaError_t moe_route_launch(const MoeRouteArgs& a, int T, cudaStream_t s) {
 
 // One CTA: histogram of the pairs by expert, tile table, placement. Which row of an expert's range a pair
 // gets depends on the order of the atomics, but every output row is computed from its own input row alone, so the
-// order changes no number.
-__global__ void __launch_bounds__(1024) moe_sort_kernel(MoeSortArgs a) {
-    griddep_launch();
-    griddep_wait();
-    extern __shared__ int ms[];
+// order changes no number. ms: [3 n_experts + 1] ints of shared memory.
+__device__ void moe_sort_cta(const MoeSortArgs& a, int* ms) {
     int* count = ms;                       // [n_experts]
     int* offset = count + a.n_experts;     // [n_experts + 1]
     int* cursor = offset + a.n_experts + 1;
@@ -167,10 +164,42 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(MoeSortArgs a) {
         a.pos[p] = row;
     }
 }
+__global__ void __launch_bounds__(1024) moe_sort_kernel(MoeSortArgs a) {
+    griddep_launch();
+    griddep_wait();
+    extern __shared__ int ms[];
+    moe_sort_cta(a, ms);
+}
 cudaError_t moe_sort_launch(const MoeSortArgs& a, cudaStream_t s) {
     const size_t smem = (size_t)(3 * a.n_experts + 1) * 4;
     if (smem > 48 * 1024) return cudaErrorInvalidValue;
     return launch_chain(moe_sort_kernel, dim3(1), dim3(1024), smem, s, a);
+}
+
+// grid (layers): the experts of the step's token ids, then (more than a few tokens) the pairs sorted into tiles
+__global__ void __launch_bounds__(1024) moe_table_kernel(const MoeTableLayer* __restrict__ layers, const int* __restrict__ tok_id, int T) {
+    griddep_launch();
+    griddep_wait();
+    extern __shared__ int ms[];
+    const MoeTableLayer l = layers[blockIdx.x];
+    const int n = T * l.top;
+    for (int p = threadIdx.x; p < n; p += blockDim.x) {
+        const int t = p / l.top;
+        l.sel[p] = l.table[(size_t)tok_id[t] * l.top + (p - t * l.top)];
+        l.tok[p] = t;
+    }
+    if (T <= MOE_FEW_TOKENS) return;
+    __syncthreads();                       // the choices are in place for the whole CTA
+    MoeSortArgs a;
+    a.sel = l.sel; a.n_pairs = n; a.top = l.top; a.n_experts = l.n_experts; a.tile = l.big_ok && n >= MOE_BIG_PAIRS ? 128 : 64;
+    a.pos = l.pos; a.x_rows = l.x_rows; a.n_tiles = l.tiles; a.tile_group = l.tiles + 1; a.tile_row0 = a.tile_group + l.max_tiles;
+    a.tile_rows = a.tile_row0 + l.max_tiles; a.max_tiles = l.max_tiles;
+    moe_sort_cta(a, ms);
+}
+cudaError_t moe_table_launch(const MoeTableLayer* dev_layers, int n_layers, int max_experts, const int* tok_id, int T, cudaStream_t s) {
+    const size_t smem = (size_t)(3 * max_experts + 1) * 4;
+    if (smem > 48 * 1024) return cudaErrorInvalidValue;
+    return launch_chain(moe_table_kernel, dim3(n_layers), dim3(1024), smem, s, dev_layers, tok_id, T);
 }
 
 // grid (T)

@@ -1,7 +1,8 @@
 // Softmax attention with a sink over the paged cache (layered.h: SinkAttnArgs): grouped query heads, sliding window, rotate-half
 // rotation of the leading entries, optional unit-RMS queries and keys, one extra term exp(sink[h]) in every head's denominator,
-// optional mixing of the heads' normalised weights across heads, sigmoid output gate. Scores, softmax, mixing and the weighted
-// sums are 32-bit; only the cache pages may be bf16.
+// optional mixing of the heads' normalised weights across heads, sigmoid output gate, optional caps on the scores; or, instead of
+// rotation and unit RMS, short convolutions and norms over whole projections. Scores, softmax, mixing and the weighted sums are
+// 32-bit; only the cache pages may be bf16.
 #include "kernels.h"
 #include "layered.h"
 #include "ptx.cuh"
@@ -28,9 +29,22 @@ __device__ __forceinline__ float sk_gate(const SinkAttnArgs& a, int t, int h, in
     if (!a.gate) return 1.f;
     return sk_sigmoid(a.gate[(size_t)t * a.ld_gate + (a.gate_per_head ? h : h * a.dv + i)]);
 }
+// the factor on a query at position pos
+__device__ __forceinline__ float sk_temperature(const SinkAttnArgs& a, int pos) {
+    return a.temp_coef != 0.f ? 1.f + a.temp_coef * logf((float)floor(((double)pos + 1.0) / a.temp_every) + 1.f) : 1.f;
+}
+// cap * tanh(s / cap) on the prompt path: below 1/8 the odd series x - x^3/3 + 2 x^5/15 (the next term is under 2.1e-7 of x), above it
+// 1 - 2 / (exp(2|x|) + 1), whose rounding errors stay near 1e-7 absolute
+__device__ __forceinline__ float sk_cap_fast(float s, float cap, float inv_cap) {
+    const float x = s * inv_cap, ax = fabsf(x), x2 = x * x;
+    const float series = fmaf(x2 * x, fmaf(x2, 2.f / 15.f, -1.f / 3.f), x);
+    const float big = copysignf(1.f - __fdividef(2.f, __expf(2.f * ax) + 1.f), x);
+    return cap * (ax < 0.125f ? series : big);
+}
 }  // namespace
 
 constexpr int SK_MAXE = 8;       // key and value sizes <= 256
+constexpr int SK_FEW_TOKENS = 8;
 
 // grid (T), 8 warps: a warp per head vector of q (H of them) and of k (G): rotation, optional unit RMS, q into scratch and k into
 // its page; then the values into theirs.
@@ -62,7 +76,8 @@ __global__ void __launch_bounds__(256) sink_attn_store_kernel(SinkAttnArgs a, Ra
             v[e] = o;
             ss = fmaf(o, o, ss);
         }
-        const float mul = a.unit_qk ? 1.f / sqrtf(warp_sum(ss) / (float)d + a.eps) : 1.f;
+        float mul = a.unit_qk ? 1.f / sqrtf(warp_sum(ss) / (float)d + a.eps) : 1.f;
+        if (is_q) mul *= sk_temperature(a, pos);
 #pragma unroll
         for (int e = 0; e < SK_MAXE; e++) {
             const int i = lane + 32 * e;
@@ -77,7 +92,163 @@ __global__ void __launch_bounds__(256) sink_attn_store_kernel(SinkAttnArgs a, Ra
         sk_store(a.v_pool, a.cache_f32, ((page * a.G + g) * a.block_tokens + in_page) * a.dv + c, row[a.v_off + i]);
     }
 }
+// ---------------------------------------------------------------- preparation with convolutions and whole-projection norms
+// grid (token groups, parts), NT threads. Part 0 = queries, 1 = keys, 2 = values, 3 = side columns: the parts share nothing, so a
+// decoded token is ready after the longest of them. A CTA takes up to TB neighbouring tokens of a segment: a thread walks its
+// channels, reads every projected row once for all TB outputs, and the rows wait in shared memory ([TB][channels], norms only) for
+// the sums of squares over all heads. Two grids:
+//   by tiles (prompts)          group = TB rows of a 64-row tile; the convolution state is moved on by a launch of its own afterwards
+//   by segments (few tokens)    group = a whole segment, TB tokens at a time; each thread then moves its channels' state on itself
+// Outputs are sums over the taps in tap order, the same in both.
+template <int TAPS>
+__device__ __forceinline__ float sk_conv(const SinkAttnArgs& a, const float* col, const float* w, int taps, int t, int i, const float* st, int C) {
+    const int n = TAPS > 0 ? TAPS : taps;
+    float acc = 0.f;
+#pragma unroll
+    for (int j = 0; j < n; j++) {
+        const int back = n - 1 - j;               // the input `back` tokens ago; before the step: the slot's last n - 1 inputs
+        const float v = i >= back ? col[(size_t)(t - back) * a.ldp] : st[(size_t)(n - 1 + i - back) * C];
+        acc = fmaf(w[j], v, acc);
+    }
+    return acc;
+}
+
+template <int NT, int TB, int TAPS>
+__global__ void __launch_bounds__(NT) sink_attn_prepare_kernel(SinkAttnArgs a, RaggedDev r, int by_segment) {
+    griddep_launch();
+    griddep_wait();
+    extern __shared__ float pr_row[];                         // [TB][n]
+    __shared__ float red[TB][33];
+    const int part = blockIdx.y, nqd = a.H * a.d, nkd = a.G * a.d, nvd = a.G * a.dv, C = nqd + nkd + nvd;
+    int seg, g0, g1;
+    if (by_segment) {
+        seg = blockIdx.x; g0 = r.seg_start[seg]; g1 = g0 + r.seg_len[seg];
+    } else {
+        constexpr int PER = 64 / TB;
+        const int tile = blockIdx.x / PER;
+        seg = r.tile_seg[tile];
+        g0 = r.tile_row0[tile] + (blockIdx.x % PER) * TB;
+        g1 = min(g0 + TB, r.seg_start[seg] + r.seg_len[seg]);
+        if (g0 >= g1) return;
+    }
+    const int start = r.seg_start[seg], slot = r.seg_slot[seg];
+    if (part == 3) {
+        for (int t = g0; t < g1; t++) {
+            const float* row = a.proj + (size_t)t * a.ldp;
+            const float gate = a.side_gate >= 0 ? sk_sigmoid(row[a.side_gate]) : 1.f;
+            for (int i = threadIdx.x; i < a.side_n; i += NT) a.out[(size_t)t * a.ld_out + a.side_col + i] = row[a.side_off + i] * gate;
+        }
+        return;
+    }
+    const int n = part == 0 ? nqd : part == 1 ? nkd : nvd, off = part == 0 ? a.q_off : part == 1 ? a.k_off : a.v_off;
+    const int ch0 = part == 0 ? 0 : part == 1 ? nqd : nqd + nkd, dd = part == 2 ? a.dv : a.d;
+    const float* nw = part == 0 ? a.q_norm_w : part == 1 ? a.k_norm_w : nullptr;
+    const int* table = a.block_tables[slot];
+    const float* state = a.conv_state ? a.conv_state + (size_t)slot * (a.taps - 1) * C + ch0 : nullptr;
+    for (int t0 = g0; t0 < g1; t0 += TB) {
+        const int nt = min(TB, g1 - t0), i0 = t0 - start;
+        size_t base[TB];                                      // of the token's row in the page (keys, values)
+        float mul[TB];
+#pragma unroll
+        for (int u = 0; u < TB; u++) {
+            const int t = min(t0 + u, g1 - 1), pos = r.tok_pos[t];
+            base[u] = ((size_t)table[pos / a.block_tokens] * a.G * a.block_tokens + pos % a.block_tokens) * dd;
+            mul[u] = part == 0 ? sk_temperature(a, pos) : 1.f;
+        }
+        auto put = [&](int u, int c, float v) {
+            if (part == 0) { a.q_rot[(size_t)(t0 + u) * nqd + c] = v; return; }
+            const int g = c / dd;
+            sk_store(part == 1 ? a.k_pool : a.v_pool, a.cache_f32, base[u] + (size_t)g * a.block_tokens * dd + (c - g * dd), v);
+        };
+        float ss[TB];
+#pragma unroll
+        for (int u = 0; u < TB; u++) ss[u] = 0.f;
+        for (int c = threadIdx.x; c < n; c += NT) {
+            const float* col = a.proj + off + c;
+            float w[TAPS > 0 ? TAPS : 1];
+            if (TAPS > 1)
+#pragma unroll
+                for (int j = 0; j < TAPS; j++) w[j] = a.conv_w[(size_t)(ch0 + c) * TAPS + j];
+#pragma unroll
+            for (int u = 0; u < TB; u++) {
+                if (u >= nt) continue;
+                float v;
+                if (!a.conv_w) v = col[(size_t)(t0 + u) * a.ldp];
+                else if (TAPS > 1) v = sk_conv<TAPS>(a, col, w, TAPS, t0 + u, i0 + u, state + c, C);
+                else v = sk_conv<0>(a, col, a.conv_w + (size_t)(ch0 + c) * a.taps, a.taps, t0 + u, i0 + u, state + c, C);
+                if (nw) { pr_row[u * n + c] = v; ss[u] = fmaf(v, v, ss[u]); }
+                else put(u, c, v * mul[u]);
+            }
+        }
+        if (nw) {
+            __syncthreads();                                  // nobody still reads the sums of the group before
+#pragma unroll
+            for (int u = 0; u < TB; u++) {
+                const float s = warp_sum(ss[u]);
+                if ((threadIdx.x & 31) == 0) red[u][threadIdx.x >> 5] = s;
+            }
+            __syncthreads();
+#pragma unroll
+            for (int u = 0; u < TB; u++) {
+                float tot = 0.f;
+#pragma unroll
+                for (int k = 0; k < NT / 32; k++) tot += red[u][k];
+                mul[u] *= 1.f / sqrtf(tot / (float)n + a.eps);
+            }
+            for (int c = threadIdx.x; c < n; c += NT) {       // a thread reads back what it wrote itself
+                const float wv = nw[c];
+#pragma unroll
+                for (int u = 0; u < TB; u++) if (u < nt) put(u, c, pr_row[u * n + c] * mul[u] * wv);
+            }
+        }
+    }
+    if (by_segment && a.conv_w && a.taps > 1) {               // entry k of the new state is read at k + len > k of the old one before it is written
+        const int hist = a.taps - 1, len = g1 - g0;
+        for (int c = threadIdx.x; c < n; c += NT) {
+            float* st = a.conv_state + (size_t)slot * hist * C + ch0 + c;
+            for (int k = 0; k < hist; k++) {
+                const int src = len + k - hist;
+                st[(size_t)k * C] = src >= 0 ? a.proj[(size_t)(g0 + src) * a.ldp + off + c] : st[(size_t)(k + len) * C];
+            }
+        }
+    }
+}
+
+template <int NT, int TB>
+static cudaError_t sink_attn_prepare_pick(const SinkAttnArgs& a, const RaggedDev& r, dim3 grid, size_t smem, int by_segment, cudaStream_t s) {
+    static bool attr_done = false;
+    if (!attr_done) {
+        cudaFuncSetAttribute(sink_attn_prepare_kernel<NT, TB, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        cudaFuncSetAttribute(sink_attn_prepare_kernel<NT, TB, 3>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        cudaFuncSetAttribute(sink_attn_prepare_kernel<NT, TB, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        attr_done = true;
+    }
+    if (a.conv_w && a.taps == 3) return launch_chain(sink_attn_prepare_kernel<NT, TB, 3>, grid, dim3(NT), smem, s, a, r, by_segment);
+    if (a.conv_w && a.taps == 4) return launch_chain(sink_attn_prepare_kernel<NT, TB, 4>, grid, dim3(NT), smem, s, a, r, by_segment);
+    return launch_chain(sink_attn_prepare_kernel<NT, TB, 0>, grid, dim3(NT), smem, s, a, r, by_segment);
+}
+
+bool sink_attn_prepares(const SinkAttnArgs& a) { return a.q_norm_w || a.k_norm_w || a.conv_w || a.side_n > 0; }
+
+static cudaError_t sink_attn_prepare_launch(const SinkAttnArgs& a, const RaggedDev& r, cudaStream_t s) {
+    if (a.rot.rot_dims > 0 || a.unit_qk) return cudaErrorInvalidValue;
+    const unsigned parts = a.side_n > 0 ? 4 : 3;
+    const size_t row = a.q_norm_w || a.k_norm_w ? (size_t)a.H * a.d * 4 : 0;         // H >= G: the query row is the longer one
+    if (row > 200 * 1024) return cudaErrorInvalidValue;
+    if (r.T <= SK_FEW_TOKENS) {
+        if ((size_t)a.H * a.d >= 1024) return sink_attn_prepare_pick<1024, 1>(a, r, dim3(r.n_seg, parts), row, 1, s);
+        return sink_attn_prepare_pick<256, 1>(a, r, dim3(r.n_seg, parts), row, 1, s);
+    }
+    cudaError_t e = 4 * row <= 100 * 1024 ? sink_attn_prepare_pick<256, 4>(a, r, dim3(r.n_tiles * 16, parts), 4 * row, 0, s)
+                                          : sink_attn_prepare_pick<256, 1>(a, r, dim3(r.n_tiles * 64, parts), row, 0, s);
+    if (e != cudaSuccess || !a.conv_w || a.taps <= 1) return e;
+    ConvArgs cv = {};
+    cv.in = a.proj + a.q_off; cv.ld_in = a.ldp; cv.C = a.H * a.d + a.G * (a.d + a.dv); cv.taps = a.taps; cv.state = a.conv_state;
+    return causal_conv_advance_launch(cv, r, s);
+}
+
 cudaError_t sink_attn_store_launch(const SinkAttnArgs& a, const RaggedDev& r, cudaStream_t s) {
+    if (sink_attn_prepares(a)) return sink_attn_prepare_launch(a, r, s);
     if (a.d > SK_MAXE * 32 || a.rot.rot_dims > a.d || a.rot.rot_dims % 2) return cudaErrorInvalidValue;
     return launch_chain(sink_attn_store_kernel, dim3(r.T), dim3(256), 0, s, a, r);
 }
@@ -89,8 +260,8 @@ cudaError_t sink_attn_store_launch(const SinkAttnArgs& a, const RaggedDev& r, cu
 // one split the sink term joins there and the normalised result is written; with several (few-token steps: the visible keys are
 // cut into `splits` equal ranges so that a single decoded token still fills the GPU) every CTA leaves (maximum, sum, output) of
 // its range in `part` and sink_attn_merge_kernel adds them in range order.
-constexpr int SK_WARPS = 8, SK_KEYS = 4, SK_MAX_SPLITS = 16, SK_FEW_TOKENS = 8, SK_VH = 4;
-template <bool F32, int VH>
+constexpr int SK_WARPS = 8, SK_KEYS = 4, SK_MAX_SPLITS = 16, SK_VH = 4;
+template <bool F32, int VH, bool CAP>
 __global__ void __launch_bounds__(SK_WARPS * 32) sink_attn_kernel(SinkAttnArgs a, RaggedDev r) {
     griddep_launch();
     griddep_wait();
@@ -140,6 +311,9 @@ __global__ void __launch_bounds__(SK_WARPS * 32) sink_attn_kernel(SinkAttnArgs a
         for (int o = 16; o > 0; o >>= 1)
 #pragma unroll
             for (int u = 0; u < SK_KEYS; u++) sc[u] += __shfl_xor_sync(0xffffffffu, sc[u], o);
+        if constexpr (CAP)
+#pragma unroll
+            for (int u = 0; u < SK_KEYS; u++) sc[u] = a.softcap * tanhf(sc[u] / a.softcap);
         float mx = m_run;
 #pragma unroll
         for (int u = 0; u < SK_KEYS; u++) if (j0 + u <= hi) mx = fmaxf(mx, sc[u]);
@@ -266,7 +440,7 @@ __device__ __forceinline__ void sk_split_bf16(float a, float b, uint32_t& hi, ui
 }
 }  // namespace
 
-template <int DMAX, int DVMAX>
+template <int DMAX, int DVMAX, bool CAP>
 __global__ void __launch_bounds__(128) sink_attn_mma_kernel(SinkAttnArgs a, RaggedDev r) {
     griddep_launch();
     griddep_wait();
@@ -306,6 +480,7 @@ __global__ void __launch_bounds__(128) sink_attn_mma_kernel(SinkAttnArgs a, Ragg
     int qlo[2];                                    // oldest visible key of the lane's two query rows
     float m_run[2], l_run[2];
     const float sink = a.sink ? a.sink[h] : -INFINITY;
+    [[maybe_unused]] const float inv_cap = CAP ? 1.f / a.softcap : 0.f;
 #pragma unroll
     for (int q2 = 0; q2 < 2; q2++) {
         const int i = p0 + qrow[q2];
@@ -358,6 +533,7 @@ __global__ void __launch_bounds__(128) sink_attn_mma_kernel(SinkAttnArgs a, Ragg
             for (int e = 0; e < 4; e++) {
                 const int rr = qrow[e >> 1], i = p0 + rr, j = j0 + ni * 8 + 2 * tq + (e & 1);
                 const bool vis = rr < nq && j <= i && j >= qlo[e >> 1];
+                if constexpr (CAP) sacc[ni][e] = sk_cap_fast(sacc[ni][e], a.softcap, inv_cap);
                 sacc[ni][e] = vis ? sacc[ni][e] : -INFINITY;
                 mx[e >> 1] = fmaxf(mx[e >> 1], sacc[ni][e]);
             }
@@ -700,19 +876,25 @@ static bool sink_attn_mixed_launch(const SinkAttnArgs& a, const RaggedDev& r, cu
     return true;
 }
 
-template <int DMAX, int DVMAX>
+template <int DMAX, int DVMAX, bool CAP>
 static cudaError_t sink_attn_mma_pick(const SinkAttnArgs& a, const RaggedDev& r, cudaStream_t s) {
     const size_t smem = (size_t)(3 * 64 * (a.d + 8) + 64 * (a.dv + 8)) * 2;
     static bool attr_done = false;
     if (!attr_done) {
-        cudaFuncSetAttribute(sink_attn_mma_kernel<DMAX, DVMAX>, cudaFuncAttributeMaxDynamicSharedMemorySize, (3 * 64 * (DMAX + 8) + 64 * (DVMAX + 8)) * 2);
+        cudaFuncSetAttribute(sink_attn_mma_kernel<DMAX, DVMAX, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (3 * 64 * (DMAX + 8) + 64 * (DVMAX + 8)) * 2);
         attr_done = true;
     }
-    return launch_chain(sink_attn_mma_kernel<DMAX, DVMAX>, dim3(r.n_tiles, a.H * (a.talk ? a.G : 1)), dim3(128), smem, s, a, r);
+    return launch_chain(sink_attn_mma_kernel<DMAX, DVMAX, CAP>, dim3(r.n_tiles, a.H * (a.talk ? a.G : 1)), dim3(128), smem, s, a, r);
+}
+
+template <bool CAP>
+static cudaError_t sink_attn_mma_sizes(const SinkAttnArgs& a, const RaggedDev& r, cudaStream_t s) {
+    if (a.d <= 64) return a.dv <= 64 ? sink_attn_mma_pick<64, 64, CAP>(a, r, s) : sink_attn_mma_pick<64, 128, CAP>(a, r, s);
+    return a.dv <= 64 ? sink_attn_mma_pick<128, 64, CAP>(a, r, s) : sink_attn_mma_pick<128, 128, CAP>(a, r, s);
 }
 
 cudaError_t sink_attn_launch(const SinkAttnArgs& a, const RaggedDev& r, cudaStream_t s) {
-    if (a.d > SK_MAXE * 32 || a.dv > SK_MAXE * 32 || a.H % a.G) return cudaErrorInvalidValue;
+    if (a.d > SK_MAXE * 32 || a.dv > SK_MAXE * 32 || a.H % a.G || (a.talk && a.softcap > 0.f)) return cudaErrorInvalidValue;
     static const bool no_mma = getenv("B2_NO_ATTN_MMA") != nullptr;        // tuning aid: scalar attention for prompts too
     const int Gv = a.talk ? a.G : 1;
     cudaError_t e;
@@ -721,8 +903,7 @@ cudaError_t sink_attn_launch(const SinkAttnArgs& a, const RaggedDev& r, cudaStre
         // with one or two key/value heads the separate sums cost no more than the second score pass and the scratch traffic
         // (measured at 8 heads over 2: 0.84 against 1.08 ms for four layers and 2048 tokens)
         if (a.talk && a.G >= 3 && !no_mixed && sink_attn_mixed_launch(a, r, s, e)) return e;
-        if (a.d <= 64) e = a.dv <= 64 ? sink_attn_mma_pick<64, 64>(a, r, s) : sink_attn_mma_pick<64, 128>(a, r, s);
-        else e = a.dv <= 64 ? sink_attn_mma_pick<128, 64>(a, r, s) : sink_attn_mma_pick<128, 128>(a, r, s);
+        e = a.softcap > 0.f ? sink_attn_mma_sizes<true>(a, r, s) : sink_attn_mma_sizes<false>(a, r, s);
     } else {
         // few tokens: enough key ranges to fill the GPU; the count depends on the step's shape and the window only, never on the
         // positions, so that a captured step can be replayed
@@ -735,13 +916,17 @@ cudaError_t sink_attn_launch(const SinkAttnArgs& a, const RaggedDev& r, cudaStre
         if (a.talk) {
             const dim3 grid(r.T, a.H * ((a.G + SK_VH - 1) / SK_VH), splits);
             const size_t smem = (size_t)SK_WARPS * SK_VH * SK_MAXE * 32 * 4;
-            e = a.cache_f32 ? launch_chain(sink_attn_kernel<true, SK_VH>, grid, dim3(SK_WARPS * 32), smem, s, a, r)
-                            : launch_chain(sink_attn_kernel<false, SK_VH>, grid, dim3(SK_WARPS * 32), smem, s, a, r);
+            e = a.cache_f32 ? launch_chain(sink_attn_kernel<true, SK_VH, false>, grid, dim3(SK_WARPS * 32), smem, s, a, r)
+                            : launch_chain(sink_attn_kernel<false, SK_VH, false>, grid, dim3(SK_WARPS * 32), smem, s, a, r);
         } else {
             const dim3 grid(r.T, a.H, splits);
             const size_t smem = (size_t)SK_WARPS * SK_MAXE * 32 * 4;
-            e = a.cache_f32 ? launch_chain(sink_attn_kernel<true, 1>, grid, dim3(SK_WARPS * 32), smem, s, a, r)
-                            : launch_chain(sink_attn_kernel<false, 1>, grid, dim3(SK_WARPS * 32), smem, s, a, r);
+            if (a.softcap > 0.f)
+                e = a.cache_f32 ? launch_chain(sink_attn_kernel<true, 1, true>, grid, dim3(SK_WARPS * 32), smem, s, a, r)
+                                : launch_chain(sink_attn_kernel<false, 1, true>, grid, dim3(SK_WARPS * 32), smem, s, a, r);
+            else
+                e = a.cache_f32 ? launch_chain(sink_attn_kernel<true, 1, false>, grid, dim3(SK_WARPS * 32), smem, s, a, r)
+                                : launch_chain(sink_attn_kernel<false, 1, false>, grid, dim3(SK_WARPS * 32), smem, s, a, r);
         }
         if (e == cudaSuccess && splits > 1) e = launch_chain(sink_attn_merge_kernel, dim3(r.T, a.H * Gv), dim3(128), 0, s, a, splits);
     }

@@ -18,11 +18,12 @@ B2_TYPE_F32, B2_TYPE_F16, B2_TYPE_I32, B2_TYPE_BF16 = 0, 1, 26, 30
 B2_MIX_WINDOW_SCAN, B2_MIX_MATRIX_MEMORY, B2_MIX_LATENT_ATTN, B2_MIX_DELTA_RULE, B2_MIX_SSD, B2_MIX_CHUNK_LINEAR = 1, 2, 3, 4, 5, 6
 B2_MIX_SINK_DELTA, B2_MIX_SINK_ATTN = 7, 8
 B2_FF_RELU2, B2_FF_MOE, B2_FF_GLU, B2_FF_PIECEWISE = 0, 1, 2, 3
-B2_EXPERT_SILU, B2_EXPERT_CLAMPED = 0, 1
+B2_EXPERT_SILU, B2_EXPERT_CLAMPED, B2_EXPERT_RELU2 = 0, 1, 2
 B2_ACT_SILU, B2_ACT_GELU_TANH = 0, 1
 B2_ATTN_BIAS, B2_ATTN_UNIT_QK, B2_ATTN_TALK, B2_ATTN_HEAD_GATE, B2_ATTN_NO_GATE, B2_ATTN_NO_SINK, B2_ATTN_ROT_PAIRS = 1, 2, 4, 8, 16, 32, 64
-B2_ROUTE_SOFTMAX_ALL, B2_ROUTE_TOPK_SOFTMAX, B2_ROUTE_SIGMOID = 0, 1, 2
-B2_BLOCK_POSTSUM_LN, B2_BLOCK_PRENORM_RMS, B2_BLOCK_OUTNORM_RMS, B2_BLOCK_HYPER_RMS, B2_BLOCK_PARALLEL_LN = 0, 1, 2, 3, 4
+B2_ATTN_CONV, B2_ATTN_FULL_NORM, B2_ATTN_UNIT_SINK, B2_ATTN_OUT_BIAS = 128, 256, 512, 1024
+B2_ROUTE_SOFTMAX_ALL, B2_ROUTE_TOPK_SOFTMAX, B2_ROUTE_SIGMOID, B2_ROUTE_TABLE = 0, 1, 2, 3
+B2_BLOCK_POSTSUM_LN, B2_BLOCK_PRENORM_RMS, B2_BLOCK_OUTNORM_RMS, B2_BLOCK_HYPER_RMS, B2_BLOCK_PARALLEL_LN, B2_BLOCK_PARALLEL_ONE_LN = 0, 1, 2, 3, 4, 5
 B2_STEP_MAX_ENTRIES = 64
 
 
@@ -44,7 +45,7 @@ class B2LayerDesc(ctypes.Structure):
         ("moe_scale", c_double), ("moe_route", c_int32), ("moe_shared_ff", c_int32), ("attn_vdim", c_int32), ("pad2_", c_int32),
         ("softcap", c_double), ("branch_scale", c_double * 2)] + [
         (n, c_int32) for n in ("attn_flags", "weights_of", "moe_expert", "moe_renorm")] + [("moe_limit", c_double), ("moe_alpha", c_double)] + [
-        (n, c_int32) for n in ("ff_act", "moe_scale_input", "la_q_rank", "kv_from")]
+        (n, c_int32) for n in ("ff_act", "moe_scale_input", "la_q_rank", "kv_from", "loop_pass", "moe_shared_gate")] + [("qtemp_coef", c_double), ("qtemp_every", c_double)]
 
 
 class B2LayeredConfig(ctypes.Structure):
@@ -52,7 +53,8 @@ class B2LayeredConfig(ctypes.Structure):
         (n, c_int32) for n in ("n_ctx", "max_seqs", "kv_block_tokens", "kv_num_blocks", "max_step_tokens", "device", "flags",
                                "block_style")] + [("logit_scale", c_float), ("embed_scale", c_float), ("norm_groups", c_int32),
                                                   ("tie_head", c_int32), ("n_streams", c_int32), ("canon_taps", c_int32),
-                                                  ("bigram_buckets", c_int32), ("bigram_mul_prev", c_int32), ("bigram_mul_cur", c_int32)]
+                                                  ("bigram_buckets", c_int32), ("bigram_mul_prev", c_int32), ("bigram_mul_cur", c_int32),
+                                                  ("embed_sinusoid", c_int32), ("loop_times", c_int32)]
 
 
 class B2Sampling(ctypes.Structure):

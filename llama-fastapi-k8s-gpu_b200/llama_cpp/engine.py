@@ -294,17 +294,18 @@ class LayeredEngine(EngineBase):
                                     getattr(dims, "block_style", 0), getattr(dims, "logit_scale", 1.0), getattr(dims, "embed_scale", 1.0),
                                     getattr(dims, "norm_groups", 1), 1 if getattr(dims, "tie_head", False) else 0,
                                     getattr(dims, "n_streams", 1), getattr(dims, "canon_taps", 0),
-                                    *getattr(dims, "bigram", (0, 0, 0)))
+                                    *getattr(dims, "bigram", (0, 0, 0)), 1 if getattr(dims, "embed_sinusoid", False) else 0,
+                                    getattr(dims, "loop_times", 0))
         descs = (_cabi.B2LayerDesc * dims.n_layer)(*dims.layers)
         h = ctypes.c_void_p()
         check(self.lib.b2_engine_create_layered(ctypes.byref(cfg), descs, ctypes.byref(h)), "b2_engine_create_layered")
         self._h = h
         self.lock = threading.RLock()
-        type_ids = {"BF16": _cabi.B2_TYPE_BF16, "F32": _cabi.B2_TYPE_F32}
+        type_ids = {"BF16": _cabi.B2_TYPE_BF16, "F32": _cabi.B2_TYPE_F32, "I32": _cabi.B2_TYPE_I32}
         try:
             for name, t in tensors.items():
                 if t.dtype not in type_ids:
-                    raise ValueError(f"tensor {name}: dtype {t.dtype} is not supported (BF16 or F32)")
+                    raise ValueError(f"tensor {name}: dtype {t.dtype} is not supported (BF16, F32, or I32 tables)")
                 shape = tuple(t.shape)
                 ne0 = shape[-1] if shape else 1
                 ne1 = int(np.prod(shape[:-1])) if len(shape) > 1 else 1

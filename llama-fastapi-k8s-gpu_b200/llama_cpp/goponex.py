@@ -36,6 +36,8 @@ class LayeredDims:
     n_streams: int = 1
     canon_taps: int = 0
     bigram: Tuple[int, int, int] = (0, 0, 0)      # buckets (0: none), factors of the previous and the current token, mod buckets
+    embed_sinusoid: bool = False
+    loop_times: int = 0                           # passes over a repeated run that start with a map of the stream and the embedding
 
 
 def _need(d: dict, key: str, where: str):

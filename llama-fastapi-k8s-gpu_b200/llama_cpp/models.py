@@ -46,7 +46,7 @@ def architectures() -> List[str]:
 
 
 def _load_builtin():
-    from . import dibesun, fazovik, goponex, llama_family, nafelix, vazunex  # noqa: F401  (each registers itself on import)
+    from . import dibesun, fazovik, goponex, llama_family, nafelix, vazunex, zogurax  # noqa: F401  (each registers itself on import)
 
 
 def open_model(path: str) -> ModelSource:
