@@ -26,7 +26,8 @@ struct DenseDev {
     const float* bias;
     float* y; int ldy;
     int T, N, K, epi;
-    int n_act;                     // EPI_BIAS_TAIL_RELU2: first column of the tail
+    int n_act, n_act_end;          // EPI_BIAS_PART_RELU2
+    __nv_bfloat16* yb;             // large-tile kernel: rounded output instead of y, or null
     float scale, p0, p1;
     const float* aux; int ldaux, aux_ns;      // aux column of output column n: n * aux_ns
     long x_bs, w_bs, y_bs, aux_bs;
@@ -68,8 +69,8 @@ __device__ __forceinline__ float gelu_tanh_act(float z) { return 0.5f * z * (1.f
 template <int EPI>
 __device__ __forceinline__ float epi_value(const DenseDev& a, const float* aux, int t, int n, float v) {
     const int epi = EPI >= 0 ? EPI : a.epi;
-    if (epi == EPI_BIAS || epi == EPI_BIAS_RELU2 || epi == EPI_BIAS_TAIL_RELU2) { if (a.bias) v += a.bias[n]; }
-    if (epi == EPI_BIAS_RELU2 || (epi == EPI_BIAS_TAIL_RELU2 && n >= a.n_act)) { v = fmaxf(v, 0.f); v = v * v; }
+    if (epi == EPI_BIAS || epi == EPI_BIAS_RELU2 || epi == EPI_BIAS_PART_RELU2) { if (a.bias) v += a.bias[n]; }
+    if (epi == EPI_BIAS_RELU2 || (epi == EPI_BIAS_PART_RELU2 && n >= a.n_act && n < a.n_act_end)) { v = fmaxf(v, 0.f); v = v * v; }
     if (epi == EPI_MUL_SIGMOID) v *= 1.f / (1.f + expf(-aux[(size_t)t * a.ldaux + n * a.aux_ns]));
     if (epi == EPI_PIECEWISE) v = v > 0.f ? fmaf(a.p0 * v, v, 0.5f * v) : fmaf(a.p1, expm1f(v) - v, 0.5f * v);
     return v * a.scale;
@@ -80,7 +81,7 @@ __device__ __forceinline__ void epi_store(const DenseDev& a, float* y, const flo
 }
 // two neighbouring columns n (even) and n + 1; rs: scales of the product rows (GLU epilogues) or null; vec2: pairs of y are
 // 8-byte aligned
-template <int EPI = -1>
+template <int EPI = -1, bool ROUNDED = false>
 __device__ __forceinline__ void epi_store2(const DenseDev& a, float* y, const float* aux, const float* rs, int t, int n, float v0, float v1,
                                            bool vec2 = false) {
     const int epi = EPI >= 0 ? EPI : a.epi;
@@ -92,7 +93,14 @@ __device__ __forceinline__ void epi_store2(const DenseDev& a, float* y, const fl
             const float g = fminf(v0, a.p0), u = fminf(fmaxf(v1, -a.p0), a.p0);
             v = g / (1.f + expf(-a.p1 * g)) * (u + 1.f);
         } else v = (epi == EPI_GLU_SILU ? silu_act(v0) : gelu_tanh_act(v0)) * v1;
-        y[(size_t)t * a.ldy + (n >> 1)] = v * a.scale;
+        if constexpr (ROUNDED) a.yb[(size_t)t * a.ldy + (n >> 1)] = __float2bfloat16(v * a.scale);
+        else y[(size_t)t * a.ldy + (n >> 1)] = v * a.scale;
+        return;
+    }
+    if constexpr (ROUNDED) {
+        __nv_bfloat16* out = a.yb + (size_t)t * a.ldy + n;
+        if (n < a.N) out[0] = __float2bfloat16(epi_value<EPI>(a, aux, t, n, v0));
+        if (n + 1 < a.N) out[1] = __float2bfloat16(epi_value<EPI>(a, aux, t, n + 1, v1));
         return;
     }
     float* dst = y + (size_t)t * a.ldy + n;
@@ -375,7 +383,7 @@ __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* smem_s
 
 constexpr int BIG_BM = 128, BIG_BN = 128, BIG_BK = 64, BIG_LD = BIG_BK + 8, BIG_STAGES = 3;
 constexpr int BIG_SMEM = BIG_STAGES * (BIG_BM + BIG_BN) * BIG_LD * 2;
-template <int EPI>
+template <int EPI, bool ROUNDED = false>
 __global__ void __launch_bounds__(256, 2) dense_mma_big_kernel(const __nv_bfloat16* __restrict__ xb, int ldxb, DenseDev a) {
     griddep_launch();
     griddep_wait();
@@ -449,8 +457,18 @@ __global__ void __launch_bounds__(256, 2) dense_mma_big_kernel(const __nv_bfloat
 #pragma unroll
             for (int e = 0; e < 4; e += 2) {
                 const int t = t0 + wm + mi * 16 + g + (e >> 1) * 8;
-                if (t < T) epi_store2<EPI>(a, y, aux, a.g.row_scale, t, n0 + wn + ni * 8 + 2 * tq, acc[mi][ni][e], acc[mi][ni][e + 1], vec2);
+                if (t < T) epi_store2<EPI, ROUNDED>(a, y, aux, a.g.row_scale, t, n0 + wn + ni * 8 + 2 * tq, acc[mi][ni][e], acc[mi][ni][e + 1], vec2);
             }
+}
+
+// The large-tile kernel reads a rounded copy of the input: [T][K]; batched: [T][x_span] with batch b at column b * x_bs; grouped
+// (128-row tiles): [x_total_rows][K], gathered by the kernel.
+bool dense_takes_rounded(const DenseArgs& a) {
+    const int span = a.batch > 1 ? a.x_span : a.K;
+    const bool tiled = a.groups && a.groups->tile_group;
+    const bool ok = a.w_type == T_BF16 && !a.exact && a.xb && a.K % 8 == 0 && (reinterpret_cast<uintptr_t>(a.w) & 15) == 0 && span % 8 == 0 &&
+                    (a.batch == 1 || (a.x_span > 0 && a.x_bs % 8 == 0 && a.w_bs % 8 == 0));
+    return ok && (a.groups ? tiled && a.groups->tile_max == BIG_BM : a.T >= 64);
 }
 
 cudaError_t dense_launch(const DenseArgs& a, cudaStream_t s) {
@@ -461,7 +479,7 @@ cudaError_t dense_launch(const DenseArgs& a, cudaStream_t s) {
     const bool wb = a.w_type == T_BF16;
     DenseDev d = {};
     d.x = a.x; d.ldx = a.ldx; d.w = a.w; d.bias = a.bias; d.y = a.y; d.ldy = a.ldy; d.T = a.T; d.N = a.N; d.K = a.K; d.epi = a.epi;
-    d.n_act = a.n_act; d.scale = a.scale; d.p0 = a.p0; d.p1 = a.p1; d.aux = a.aux; d.ldaux = a.ldaux; d.aux_ns = a.aux_one ? 0 : 1; d.x_bs = a.x_bs; d.w_bs = a.w_bs; d.y_bs = a.y_bs; d.aux_bs = a.aux_bs;
+    d.n_act = a.n_act; d.n_act_end = a.n_act_end; d.yb = a.y_rounded; d.scale = a.scale; d.p0 = a.p0; d.p1 = a.p1; d.aux = a.aux; d.ldaux = a.ldaux; d.aux_ns = a.aux_one ? 0 : 1; d.x_bs = a.x_bs; d.w_bs = a.w_bs; d.y_bs = a.y_bs; d.aux_bs = a.aux_bs;
     if (a.groups) { d.g = *a.groups; d.grouped = a.groups->tile_group ? 2 : 1; }
     if (d.grouped == 1 || (!d.grouped && a.T <= ROWS_MAX_T)) return wb ? launch_rows<__nv_bfloat16>(d, a.batch, s) : launch_rows<float>(d, a.batch, s);
     // few output columns in 32-bit (router scores): the tiled kernel would run a handful of CTAs over the whole K; the
@@ -478,30 +496,42 @@ cudaError_t dense_launch(const DenseArgs& a, cudaStream_t s) {
         return wb ? launch_rows<__nv_bfloat16>(c, 1, s) : launch_rows<float>(c, 1, s);
     }
     const unsigned gz = d.grouped ? 1 : a.batch;
-    // The large-tile kernel reads a rounded copy of the input: [T][K]; batched: [T][x_span] with batch b at column b * x_bs;
-    // grouped (128-row tiles): [x_total_rows][K], gathered by the kernel.
     const int x_rows_total = d.grouped ? a.groups->x_total_rows : a.T;
     const int span = a.batch > 1 ? a.x_span : a.K;
-    const bool big_ok = wb && !a.exact && a.xb && a.K % 8 == 0 && (reinterpret_cast<uintptr_t>(a.w) & 15) == 0 && span % 8 == 0 &&
-                        (a.batch == 1 || (a.x_span > 0 && a.x_bs % 8 == 0 && a.w_bs % 8 == 0));
-    if (d.grouped == 2 && a.groups->tile_max == BIG_BM && !big_ok) return cudaErrorInvalidValue;
-    if (big_ok && (d.grouped ? a.groups->tile_max == BIG_BM : a.T >= 64)) {
+    const bool big = dense_takes_rounded(a);
+    if ((d.grouped == 2 && a.groups->tile_max == BIG_BM && !big) || (!big && (a.x_rounded || a.y_rounded))) return cudaErrorInvalidValue;
+    if (big) {
         static const auto kernels = [] {
             std::array<void (*)(const __nv_bfloat16*, int, DenseDev), 9> k = {
                 dense_mma_big_kernel<EPI_NONE>, dense_mma_big_kernel<EPI_BIAS>, dense_mma_big_kernel<EPI_BIAS_RELU2>, dense_mma_big_kernel<EPI_GLU_SILU>,
                 dense_mma_big_kernel<EPI_MUL_SIGMOID>, dense_mma_big_kernel<EPI_GLU_CLAMP>, dense_mma_big_kernel<EPI_PIECEWISE>, dense_mma_big_kernel<EPI_GLU_GELU>,
-                dense_mma_big_kernel<EPI_BIAS_TAIL_RELU2>};
+                dense_mma_big_kernel<EPI_BIAS_PART_RELU2>};
             for (auto f : k) cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, BIG_SMEM);
             return k;
         }();
         if (a.epi < 0 || a.epi >= (int)kernels.size()) return cudaErrorInvalidValue;
-        const long pairs = (long)x_rows_total * (span / 2);
-        cudaError_t ce = launch_chain(rows_to_bf16_kernel, dim3((unsigned)std::min<long>((pairs + 255) / 256, 148 * 8)), dim3(256), 0, s,
-                                      a.x, a.ldx, x_rows_total, span, a.xb);
-        if (ce != cudaSuccess) return ce;
+        const __nv_bfloat16* xb = a.x_rounded;
+        if (!xb) {
+            const long pairs = (long)x_rows_total * (span / 2);
+            const cudaError_t ce = launch_chain(rows_to_bf16_kernel, dim3((unsigned)std::min<long>((pairs + 255) / 256, 148 * 8)), dim3(256), 0, s,
+                                                a.x, a.ldx, x_rows_total, span, a.xb);
+            if (ce != cudaSuccess) return ce;
+            xb = a.xb;
+        }
         const unsigned gy = d.grouped ? (unsigned)a.groups->max_tiles : (unsigned)((a.T + BIG_BM - 1) / BIG_BM);
-        return launch_chain(kernels[a.epi], dim3((a.N + BIG_BN - 1) / BIG_BN, gy, gz), dim3(256), (size_t)BIG_SMEM, s,
-                            (const __nv_bfloat16*)a.xb, span, d);
+        auto kernel = kernels[a.epi];
+        if (a.y_rounded) {             // outputs that only feed the next product: the activations of experts
+            static const auto rounded = [] {
+                std::array<void (*)(const __nv_bfloat16*, int, DenseDev), 3> k = {
+                    dense_mma_big_kernel<EPI_BIAS_RELU2, true>, dense_mma_big_kernel<EPI_GLU_SILU, true>, dense_mma_big_kernel<EPI_GLU_CLAMP, true>};
+                for (auto f : k) cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, BIG_SMEM);
+                return k;
+            }();
+            const int which = a.epi == EPI_BIAS_RELU2 ? 0 : a.epi == EPI_GLU_SILU ? 1 : a.epi == EPI_GLU_CLAMP ? 2 : -1;
+            if (which < 0) return cudaErrorInvalidValue;
+            kernel = rounded[which];
+        }
+        return launch_chain(kernel, dim3((a.N + BIG_BN - 1) / BIG_BN, gy, gz), dim3(256), (size_t)BIG_SMEM, s, xb, span, d);
     }
     dim3 grid((a.N + 63) / 64, d.grouped ? (unsigned)a.groups->max_tiles : (unsigned)((a.T + 63) / 64), gz);
     if (wb && !a.exact) return launch_chain(dense_mma_kernel, grid, dim3(128), 0, s, d);

@@ -100,6 +100,10 @@ struct LayeredModel {
     float *xs = nullptr, *hc = nullptr, *cross = nullptr;     // copies of the stream [S][max_step_tokens][W]; convolved sublayer input; per-(query head, value head) attention sums
     float *x = nullptr, *proj = nullptr, *buf[4] = {}, *oL = nullptr, *oR = nullptr, *hn = nullptr, *hn2 = nullptr, *ff = nullptr, *rows = nullptr, *logits = nullptr;
     __nv_bfloat16* xb = nullptr;       // a product's input rounded to bf16 [max_step_tokens][widest input]
+    // blocks behind one norm: what a producer leaves already rounded for the large products: the normed row, the mixer's output row;
+    // experts' activations (every family)
+    __nv_bfloat16 *hn_b = nullptr, *mix_b = nullptr, *moe_hb = nullptr;
+    const __nv_bfloat16* hn_rounded = nullptr;      // hn_b when the step's boundary kernels fill it
     std::unordered_map<std::string, StepGraph> graphs;     // replayable small steps, by shape (b2_step)
     bool graphs_on = true;
     // mixture of experts: router outputs, choices, the sorted pair table, expert activations and outputs
@@ -337,6 +341,7 @@ int layered_finalize(b2_engine* e) {
     size_t moe_pairs = 0, moe_slots = 0, moe_ff = 0, moe_experts = 0, moe_xb = 0;     // moe_xb: expert activations per step token
     const bool hyper = c.block_style == B2_BLOCK_HYPER_RMS;
     const int n_streams = std::max(1, c.n_streams);
+    size_t max_mix = 0;                                    // mixer output row, with what rides along
     size_t max_cross = 0, max_pbuf = 0, max_part = 0;      // max_part: floats of one token's partial attention results with one key range
     // cache pages and recurrent state of a sink-attention layer (every run of a repeated layer has its own)
     auto sink_state = [&](LyLayer& L) -> int {
@@ -410,14 +415,14 @@ int layered_finalize(b2_engine* e) {
             // a gated squared-ReLU shared expert behind the same norm rides along
             const int sff = one_norm && d.n_ff > 0 && d.ff_kind == B2_FF_MOE && d.moe_expert == B2_EXPERT_RELU2 ? d.moe_shared_ff : 0;
             std::vector<std::pair<std::string, int>> parts = {{a + "q", qd}, {a + "k", kd}, {a + "v", vd}};
+            if (sff > 0) parts.push_back({p + "mlp.shared.up", sff});       // 16-byte rows first, the narrow ones last
             if (gate) parts.push_back({a + "g", gd});
             if (two) for (auto& pr : std::vector<std::pair<std::string, int>>{{b + "q", rkd}, {b + "k", rkd}, {b + "v", rvd}, {b + "b", Hr}, {b + "a", Hr}, {b + "g", rvd}}) parts.push_back(pr);
             if (sff > 0 && d.moe_shared_gate) parts.push_back({p + "mlp.shared.sg", 1});
-            if (sff > 0) parts.push_back({p + "mlp.shared.up", sff});
             std::vector<int> offs;
             if ((rc = fuse(e, m, parts, W, L.sk_proj, offs))) return rc;
-            L.q_off = offs[0]; L.k_off = offs[1]; L.v_off = offs[2]; L.gl_off = gate ? offs[3] : -1;
-            if (sff > 0) { L.su_off = offs.back(); L.sg_off = d.moe_shared_gate ? offs[offs.size() - 2] : -1; }
+            L.q_off = offs[0]; L.k_off = offs[1]; L.v_off = offs[2]; L.gl_off = gate ? offs[sff > 0 ? 4 : 3] : -1;
+            if (sff > 0) { L.su_off = offs[3]; L.sg_off = d.moe_shared_gate ? offs.back() : -1; }
             if (d.attn_flags & B2_ATTN_BIAS) {       // one bias row for the fused product; the gate has none
                 if ((rc = dev_alloc(m, (void**)&L.sk_bias, (size_t)L.sk_proj.N * 4, true))) return rc;
                 const std::pair<std::string, int> bs[3] = {{a + "q.b", qd}, {a + "k.b", kd}, {a + "v.b", vd}};
@@ -454,7 +459,8 @@ int layered_finalize(b2_engine* e) {
                 if ((rc = vec_f32(e, m, b + "out", W, 1, &L.right_w))) return rc;
             }
             if ((rc = sink_state(L))) return rc;
-            max_proj = std::max<size_t>(max_proj, L.sk_proj.N);
+            max_proj = std::max<size_t>(max_proj, (L.sk_proj.N + 3) / 4 * 4);
+            max_mix = std::max<size_t>(max_mix, (size_t)od + sff);
             max_buf = std::max<size_t>({max_buf, (size_t)qd, (size_t)od + sff, two ? (size_t)L.conv_C : 1, two ? (size_t)rvd : 1});
             if (d.attn_flags & B2_ATTN_TALK) max_cross = std::max<size_t>(max_cross, (size_t)H * G * d.attn_vdim);
             max_part = std::max<size_t>(max_part, (size_t)H * ((d.attn_flags & B2_ATTN_TALK) ? G : 1) * (d.attn_vdim + 2));
@@ -693,6 +699,10 @@ int layered_finalize(b2_engine* e) {
     max_ff = std::max(max_ff, max_glu);
     if ((rc = dev_alloc(m, (void**)&m->ff, (size_t)Tm * max_ff * 4))) return rc;
     if (!m->exact && (rc = dev_alloc(m, (void**)&m->xb, (size_t)(Tm + B2_STEP_MAX_ENTRIES) * std::max<size_t>({max_buf, max_ff, (size_t)(c.loop_times > 0 ? 2 * W : W), moe_xb}) * 2 + 64))) return rc;
+    if (one_norm && !m->exact) {
+        if ((rc = dev_alloc(m, (void**)&m->hn_b, (size_t)Tm * W * 2 + 64))) return rc;
+        if (max_mix > 0 && (rc = dev_alloc(m, (void**)&m->mix_b, (size_t)Tm * max_mix * 2 + 64))) return rc;
+    }
     if (max_part > 0) {                      // sink attention: up to 8 tokens x 16 key ranges
         m->attn_split_floats = (int)std::min<size_t>(max_part * 8 * 16, (size_t)1 << 28);
         if ((rc = dev_alloc(m, (void**)&m->attn_split, (size_t)m->attn_split_floats * 4))) return rc;
@@ -711,6 +721,7 @@ int layered_finalize(b2_engine* e) {
         if ((rc = dev_alloc(m, (void**)&m->moe_rows, moe_pairs * 4, true))) return rc;
         if ((rc = dev_alloc(m, (void**)&m->moe_tiles, (size_t)(3 * m->moe_max_tiles + 1) * 4, true))) return rc;
         if ((rc = dev_alloc(m, (void**)&m->moe_h, moe_pairs * moe_ff * 4))) return rc;
+        m->moe_hb = reinterpret_cast<__nv_bfloat16*>(m->moe_h);       // one or the other, never both in a step
         if ((rc = dev_alloc(m, (void**)&m->moe_y, moe_pairs * W * 4))) return rc;
     }
     if ((rc = dev_alloc(m, (void**)&m->rows, (size_t)LOGIT_ROWS * W * 4))) return rc;
@@ -965,6 +976,13 @@ static int dense(b2_engine* e, LayeredModel* m, const DenseW& w, const float* x,
     return B2_OK;
 }
 
+// a plain product of T rows with these weights takes inputs that are rounded already
+static bool takes_rounded(const LayeredModel* m, const DenseW& w, int T) {
+    DenseArgs a = {};
+    a.w = w.w; a.w_type = w.type; a.T = T; a.N = w.N; a.K = w.K; a.exact = m->exact; a.xb = m->xb;
+    return dense_takes_rounded(a);
+}
+
 // ---- token mixers: each reads the sublayer input `in` [T][W] and leaves its output in m->oL (the two-branch mixer also m->oR)
 static int mix_window_scan(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in) {
     const b2_layered_config& c = m->c;
@@ -1196,11 +1214,12 @@ static int mix_sink(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& 
     const b2_layered_config& c = m->c;
     const b2_layer_desc& d = L.d;
     cudaStream_t st = e->stream;
-    const int T = r.T, W = c.n_embd, Np = L.sk_proj.N, H = d.n_head, od = H * d.attn_vdim, Ko = L.attn_o.K;
+    const int T = r.T, W = c.n_embd, Np = (L.sk_proj.N + 3) / 4 * 4 /* rows start on 16 bytes */, H = d.n_head, od = H * d.attn_vdim, Ko = L.attn_o.K;
     int rc;
     DenseArgs pj = {};
-    pj.n_act = L.su_off;                   // the rows of a shared expert that rides along get their activation here
-    if ((rc = dense(e, m, L.sk_proj, in, W, m->proj, Np, T, L.sk_bias, L.su_off >= 0 ? EPI_BIAS_TAIL_RELU2 : L.sk_bias ? EPI_BIAS : EPI_NONE, 1, &pj))) return rc;
+    pj.n_act = L.su_off; pj.n_act_end = L.su_off + Ko - od;       // the rows of a shared expert that rides along get their activation here
+    if (in == m->hn) pj.x_rounded = m->hn_rounded;
+    if ((rc = dense(e, m, L.sk_proj, in, W, m->proj, Np, T, L.sk_bias, L.su_off >= 0 ? EPI_BIAS_PART_RELU2 : L.sk_bias ? EPI_BIAS : EPI_NONE, 1, &pj))) return rc;
     SinkAttnArgs a = {};
     a.proj = m->proj; a.ldp = Np; a.q_off = L.q_off; a.k_off = L.k_off; a.v_off = L.v_off;
     a.rot.cos = L.rot_cos; a.rot.sin = L.rot_sin; a.rot.rot_dims = d.rot_dims; a.unit_qk = (d.attn_flags & B2_ATTN_UNIT_QK) ? 1 : 0;
@@ -1208,19 +1227,25 @@ static int mix_sink(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& 
     a.H = H; a.G = d.n_head_kv; a.d = d.head_dim; a.dv = d.attn_vdim; a.window = d.window; a.scale = (float)d.attn_scale; a.eps = c.norm_eps;
     a.sink = L.sink; a.talk = L.talk; a.gate = L.gl_off >= 0 ? m->proj + L.gl_off : nullptr; a.ld_gate = Np; a.gate_per_head = (d.attn_flags & B2_ATTN_HEAD_GATE) ? 1 : 0;
     a.q_rot = m->buf[0]; a.cross = m->cross; a.out = m->buf[1]; a.ld_out = Ko;
-    a.softcap = (float)d.softcap; a.temp_coef = (float)d.qtemp_coef; a.temp_every = d.qtemp_every;
+    a.softcap = (float)d.softcap; a.temp_coef = (float)d.qtemp_coef; a.temp_every = (float)d.qtemp_every;
     a.q_norm_w = L.q_norm; a.k_norm_w = L.k_norm;
     if (d.attn_flags & B2_ATTN_CONV) { a.conv_w = L.st_conv_w; a.taps = d.conv_taps; a.conv_state = L.st_conv_state; }
     if (L.su_off >= 0) { a.side_off = L.su_off; a.side_gate = L.sg_off; a.side_n = Ko - od; a.side_col = od; }
     a.pbuf = m->attn_pbuf; a.pbuf_floats = m->attn_pbuf_floats;
     a.part = m->attn_split; a.part_capacity = m->attn_split_floats; a.max_keys = d.window > 0 ? std::min(d.window, c.n_ctx) : c.n_ctx;
+    DenseArgs op = {};
+    if (m->mix_b && !L.talk && sink_attn_on_tensor_cores(a, T) && (sink_attn_prepares(a) || Ko == od) && takes_rounded(m, L.attn_o, T)) {
+        a.out_bf16 = m->mix_b;
+        op.x_rounded = m->mix_b;
+    }
     {
         StepProfiler sp(m, st, 2);
         CK(sink_attn_store_launch(a, r, st));
         CK(sink_attn_launch(a, r, st));
         e->launches += L.talk ? 3 : 2;
+        if (a.conv_w && a.taps > 1 && T > 8) e->launches++;
     }
-    if ((rc = dense(e, m, L.attn_o, m->buf[1], Ko, m->oL, W, T, L.o_bias, L.o_bias ? EPI_BIAS : EPI_NONE))) return rc;
+    if ((rc = dense(e, m, L.attn_o, m->buf[1], Ko, m->oL, W, T, L.o_bias, L.o_bias ? EPI_BIAS : EPI_NONE, 1, &op))) return rc;
     if (d.mixer != B2_MIX_SINK_DELTA) return B2_OK;
     const int Hr = d.mm_heads, G = d.key_heads, kd = G * d.mm_dim, vd = Hr * d.mm_vdim;
     ConvArgs cv = {};
@@ -1330,12 +1355,17 @@ static int ff_moe(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r,
     g.x_rows = tiled ? x_rows : tok; g.w_stride = (long)L.gate_up.N * W; g.x_total_rows = T;
     up.groups = &g;
     up.p0 = (float)d.moe_limit; up.p1 = (float)d.moe_alpha;
+    if (big) {                                     // the activations only feed the down maps: left rounded
+        if (in == m->hn) up.x_rounded = m->hn_rounded;
+        up.y_rounded = m->moe_hb;
+    }
     const int act = d.moe_expert == B2_EXPERT_CLAMPED ? EPI_GLU_CLAMP : d.moe_expert == B2_EXPERT_RELU2 ? EPI_BIAS_RELU2 : EPI_GLU_SILU;
     if ((rc = dense(e, m, L.gate_up, in, W, m->moe_h, ff, pairs, nullptr, act, 1, &up))) return rc;
     DenseGroups g2 = g;
     g2.x_rows = nullptr; g2.row_scale = nullptr; g2.w_stride = (long)W * ff; g2.x_total_rows = pairs;
     DenseArgs dn = {};
     dn.groups = &g2;
+    if (big) dn.x_rounded = m->moe_hb;
     if (table) dn.scale = 1.f / (float)d.moe_top;
     if ((rc = dense(e, m, L.e_down, m->moe_h, ff, m->moe_y, W, pairs, nullptr, EPI_NONE, 1, &dn))) return rc;
     if (defer) {
@@ -1408,6 +1438,7 @@ static int run_layers(b2_engine* e, LayeredModel* m, const RaggedDev& r) {
         pending_moe = MoeJoinArgs{};
         return B2_OK;
     };
+    m->hn_rounded = nullptr;
     if (c.block_style == B2_BLOCK_HYPER_RMS) {
         // The embedding sits in copy 0. A sublayer's output waits (in m->oL / m->oR / the mixture's rows) until the next boundary:
         // one kernel writes it back into all copies, reads the next sublayer's input and norms it.
@@ -1468,6 +1499,19 @@ static int run_layers(b2_engine* e, LayeredModel* m, const RaggedDev& r) {
         // is its bias), and the norm follows.
         const bool one_norm = c.block_style == B2_BLOCK_PARALLEL_ONE_LN;
         float* ff_in = one_norm ? m->hn : m->hn2;
+        // the boundary leaves the normed row rounded when every product of the large kernel that reads it takes it so, and in 32-bit when
+        // any other kernel reads it
+        auto norms = [&](ParallelJoinArgs& p, const LyLayer& N) {
+            p.w1 = N.norm1; p.b1 = N.norm1_b; p.y1 = m->hn;
+            if (!one_norm && N.d.n_ff > 0) { p.w2 = N.norm2; p.b2 = N.norm2_b; p.y2 = m->hn2; }
+            m->hn_rounded = nullptr;
+            if (one_norm && m->hn_b && N.d.mixer == B2_MIX_SINK_ATTN && takes_rounded(m, N.sk_proj, T)) {
+                m->hn_rounded = p.y1_bf16 = m->hn_b;
+                const bool moe = N.d.n_ff > 0 && N.d.ff_kind == B2_FF_MOE;
+                const bool big = moe && T * N.d.moe_top >= MOE_BIG_PAIRS && N.gate_up.type == T_BF16 && W % 8 == 0 && N.d.n_ff % 8 == 0;
+                if (N.d.n_ff == 0 || (big && N.d.moe_route == B2_ROUTE_TABLE)) p.y1 = nullptr;
+            }
+        };
         ParallelJoinArgs pj = {};
         MoeJoinArgs pj_moe = {};
         auto boundary = [&]() -> int {
@@ -1487,10 +1531,7 @@ static int run_layers(b2_engine* e, LayeredModel* m, const RaggedDev& r) {
                     if ((rc = boundary())) return rc;
                 }
             } else {
-                if (next) {
-                    pj.w1 = next->norm1; pj.b1 = next->norm1_b; pj.y1 = m->hn;
-                    if (!one_norm && next->d.n_ff > 0) { pj.w2 = next->norm2; pj.b2 = next->norm2_b; pj.y2 = m->hn2; }
-                }
+                if (next) norms(pj, *next);
                 if ((rc = boundary())) return rc;
             }
             if (m->trace && li > 0)
@@ -1498,8 +1539,7 @@ static int run_layers(b2_engine* e, LayeredModel* m, const RaggedDev& r) {
             if (!next) break;
             if (pass) {
                 if ((rc = dense(e, m, m->loop_in, m->loop_x, 2 * W, m->x, W, T, m->loop_step + (size_t)(next->d.loop_pass - 1) * W, EPI_BIAS))) return rc;
-                pj.w1 = next->norm1; pj.b1 = next->norm1_b; pj.y1 = m->hn;
-                if (!one_norm && next->d.n_ff > 0) { pj.w2 = next->norm2; pj.b2 = next->norm2_b; pj.y2 = m->hn2; }
+                norms(pj, *next);
                 if ((rc = boundary())) return rc;
             }
             LyLayer& L = m->layers[li];

@@ -35,9 +35,9 @@ struct RaggedDev {             // device pointers, valid for one step
 // EPI_GLU_GELU: the same with the tanh form of GELU.
 // EPI_MUL_SIGMOID: the product times sigmoid(aux[t][n]) (aux_one: sigmoid(aux[t][0]) for all columns of a batch entry).
 // EPI_GLU_CLAMP: pairs as above; g = min(gate, p0), u = clamp(up, -p0, p0); output = g * sigmoid(p1 * g) * (u + 1).
-// EPI_BIAS_TAIL_RELU2: bias (if any), then columns n >= n_act through the squared ReLU (a fused matrix whose last rows feed one).
+// EPI_BIAS_PART_RELU2: bias (if any), then columns n_act <= n < n_act_end through the squared ReLU (a fused matrix of which some rows feed one).
 // EPI_PIECEWISE: z > 0: p0 z^2 + z / 2; else p1 (exp(z) - 1 - z) + z / 2.
-enum DenseEpi { EPI_NONE = 0, EPI_BIAS = 1, EPI_BIAS_RELU2 = 2, EPI_GLU_SILU = 3, EPI_MUL_SIGMOID = 4, EPI_GLU_CLAMP = 5, EPI_PIECEWISE = 6, EPI_GLU_GELU = 7, EPI_BIAS_TAIL_RELU2 = 8 };
+enum DenseEpi { EPI_NONE = 0, EPI_BIAS = 1, EPI_BIAS_RELU2 = 2, EPI_GLU_SILU = 3, EPI_MUL_SIGMOID = 4, EPI_GLU_CLAMP = 5, EPI_PIECEWISE = 6, EPI_GLU_GELU = 7, EPI_BIAS_PART_RELU2 = 8 };
 // Grouped products (mixture of experts): the rows of a step's (token, choice) pairs, each against the matrix of its group.
 //   tiles == nullptr: row p of the product is pair p itself, blockIdx.y walks the pairs one by one (few-token steps);
 //   else: pairs sorted by group, tile i = rows [tile_row0[i], + tile_rows[i]) of group tile_group[i]; *n_tiles of them.
@@ -66,15 +66,20 @@ struct DenseArgs {
     bool exact;                     // true: 32-bit multiply-adds (no tensor cores, inputs not rounded)
     __nv_bfloat16* xb;              // scratch [T][K] for X rounded to bf16 (large tensor-core steps); null: not available
     float scale = 1.f;              // the product (after the epilogue) times this
-    int n_act = 0;                  // EPI_BIAS_TAIL_RELU2
+    int n_act = 0, n_act_end = 0;   // EPI_BIAS_PART_RELU2
     float p0 = 0.f, p1 = 0.f;       // constants of EPI_GLU_CLAMP / EPI_PIECEWISE
     const float* aux = nullptr; int ldaux = 0; bool aux_one = false;      // EPI_MUL_SIGMOID
     // batch > 1: `batch` independent products, operand b at x + b * x_bs, w + b * w_bs (elements), y + b * y_bs, aux + b * aux_bs
     int batch = 1; long x_bs = 0, w_bs = 0, y_bs = 0, aux_bs = 0;
+    // products of the large tensor-core kernel (dense_takes_rounded): the input rounded to bf16 [rows][K] if the producer has left it, and
+    // the output rounded to bf16 [rows][ldy] instead of f32 for the next one
+    const __nv_bfloat16* x_rounded = nullptr;
+    __nv_bfloat16* y_rounded = nullptr;
     int x_span = 0;                 // batch > 1: columns of x that hold all batches' inputs (for the rounded copy), or 0
     const DenseGroups* groups = nullptr;            // grouped product (T = number of pair rows)
 };
 cudaError_t dense_launch(const DenseArgs& a, cudaStream_t s);
+bool dense_takes_rounded(const DenseArgs& a);          // dense_launch takes the kernel that reads rounded inputs
 
 // ---------------------------------------------------------------- mixers and norms (mixers.cu)
 // x[t] = table[tok_id[t]] * scale (+ bigram row of (tok_prev[t], tok_id[t])) (+ a sinusoid of the position)
@@ -302,6 +307,7 @@ struct ParallelJoinArgs {
     const float *w2, *b2; float* y2;
     float eps;
     float* x_copy; int ld_copy;
+    __nv_bfloat16* y1_bf16;        // the first norm's output rounded, for products that take it that way; y1 may then be null
 };
 cudaError_t parallel_join_launch(const ParallelJoinArgs& a, int W, int T, cudaStream_t s);
 
@@ -350,7 +356,7 @@ struct SinkAttnArgs {
     RotaryTable rot;                                           // pairs (i, i + rot_dims / 2)
     int unit_qk;
     float softcap;                                             // <= 0: none
-    float temp_coef; double temp_every;                        // q at position p times 1 + coef * ln(floor((p + 1) / every) + 1); coef 0: off
+    float temp_coef, temp_every;                               // q at position p times 1 + coef * ln(floor((p + 1) / every) + 1); coef 0: off
     const float* q_norm_w; const float* k_norm_w;              // [H*d], [G*d]: whole-projection norms, or null
     const float* conv_w; int taps; float* conv_state;          // [C][taps], state [slot][taps-1][C], C = H*d + G*d + G*dv; null: none
     int side_off, side_gate, side_n, side_col;                 // side_n == 0: none
@@ -367,9 +373,11 @@ struct SinkAttnArgs {
     int max_keys;                                              // most keys a query can see (the window, or the context size)
     float* pbuf; size_t pbuf_floats;                           // prompts with mixed heads: the normalised weights of a group of query tiles
     float* out; int ld_out;                                    // out[t][h*dv + i]
+    __nv_bfloat16* out_bf16;                                   // != null: rounded here instead (prompts, sink_attn_on_tensor_cores), same strides
 };
 // rotation (and unit RMS) of q and k, or the preparation above; keys and values into the pages; the convolution's state moves on
 bool sink_attn_prepares(const SinkAttnArgs& a);       // sink_attn_store_launch takes the preparation path
+bool sink_attn_on_tensor_cores(const SinkAttnArgs& a, int T);       // sink_attn_launch takes the prompt kernel
 cudaError_t sink_attn_store_launch(const SinkAttnArgs& a, const RaggedDev& r, cudaStream_t s);
 cudaError_t sink_attn_launch(const SinkAttnArgs& a, const RaggedDev& r, cudaStream_t s);
 

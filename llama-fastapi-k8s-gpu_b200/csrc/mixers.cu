@@ -42,6 +42,7 @@ __device__ __forceinline__ float softplus_f(float z) { return z > 0.f ? z + log1
 __device__ __forceinline__ float log_sigmoid_f(float z) { return -softplus_f(-z); }
 
 // ---------------------------------------------------------------- embedding, gather
+constexpr int EMBED_COLS = 512;      // columns per CTA
 template <typename TW>
 __global__ void embed_ragged_kernel(const TW* __restrict__ table, int W, const int* __restrict__ tok, float* __restrict__ x, float scale,
                                     const int* __restrict__ tok_prev, BigramTable bg, EmbedExtra ex) {
@@ -54,7 +55,8 @@ __global__ void embed_ragged_kernel(const TW* __restrict__ table, int W, const i
         const int prev = tok_prev[t];
         pair_row = prev < 0 ? bg.buckets : (size_t)(((long long)prev * bg.mul_prev + (long long)cur * bg.mul_cur) % bg.buckets);
     }
-    for (int i = threadIdx.x; i < W; i += blockDim.x) {
+    const int i1 = min(W, (int)(blockIdx.y + 1) * EMBED_COLS);
+    for (int i = blockIdx.y * EMBED_COLS + threadIdx.x; i < i1; i += blockDim.x) {
         float v;
         if constexpr (sizeof(TW) == 2) v = __bfloat162float(row[i]) * scale;
         else v = row[i] * scale;
@@ -76,8 +78,9 @@ cudaError_t embed_ragged_launch(const void* table, int w_type, int W, const int*
     const EmbedExtra ex = extra ? *extra : EmbedExtra{};
     const BigramTable bg = bigram ? *bigram : BigramTable{};
     if (bg.table && !tok_prev) return cudaErrorInvalidValue;
-    if (w_type == T_BF16) return launch_chain(embed_ragged_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, s, (const __nv_bfloat16*)table, W, tok_id, x, scale, tok_prev, bg, ex);
-    if (w_type == T_F32) return launch_chain(embed_ragged_kernel<float>, dim3(T), dim3(128), 0, s, (const float*)table, W, tok_id, x, scale, tok_prev, bg, ex);
+    const dim3 grid(T, (W + EMBED_COLS - 1) / EMBED_COLS);
+    if (w_type == T_BF16) return launch_chain(embed_ragged_kernel<__nv_bfloat16>, grid, dim3(128), 0, s, (const __nv_bfloat16*)table, W, tok_id, x, scale, tok_prev, bg, ex);
+    if (w_type == T_F32) return launch_chain(embed_ragged_kernel<float>, grid, dim3(128), 0, s, (const float*)table, W, tok_id, x, scale, tok_prev, bg, ex);
     return cudaErrorInvalidValue;
 }
 
@@ -201,14 +204,18 @@ __global__ void __launch_bounds__(NT) parallel_join_kernel(ParallelJoinDev p, in
         row[i] = v;
         sum += v;
     }
-    if (!a.y1 && !a.y2) return;
+    if (!a.w1 && !a.w2) return;
     const float mean = block_sum(sum, red) / (float)W;
     float sq = 0.f;
     for (int i = threadIdx.x; i < W; i += NT) { const float dlt = row[i] - mean; sq = fmaf(dlt, dlt, sq); }
     const float rstd = 1.f / sqrtf(block_sum(sq, red) / (float)W + a.eps);
     for (int i = threadIdx.x; i < W; i += NT) {
         const float u = (row[i] - mean) * rstd;
-        if (a.y1) a.y1[base + i] = fmaf(u, a.w1[i], a.b1 ? a.b1[i] : 0.f);
+        if (a.w1) {
+            const float v = fmaf(u, a.w1[i], a.b1 ? a.b1[i] : 0.f);
+            if (a.y1) a.y1[base + i] = v;
+            if (a.y1_bf16) a.y1_bf16[base + i] = __float2bfloat16(v);
+        }
         if (a.y2) a.y2[base + i] = fmaf(u, a.w2[i], a.b2 ? a.b2[i] : 0.f);
     }
 }

@@ -8,6 +8,7 @@
 #include "ptx.cuh"
 #include "quant_blocks.cuh"
 
+#include <cooperative_groups.h>
 #include <stdlib.h>
 
 #include <algorithm>
@@ -29,18 +30,13 @@ __device__ __forceinline__ float sk_gate(const SinkAttnArgs& a, int t, int h, in
     if (!a.gate) return 1.f;
     return sk_sigmoid(a.gate[(size_t)t * a.ld_gate + (a.gate_per_head ? h : h * a.dv + i)]);
 }
-// the factor on a query at position pos
+// the factor on a query at position pos (the rounded quotient of two integers below 2^24 never reaches an integer that the exact one
+// does not)
 __device__ __forceinline__ float sk_temperature(const SinkAttnArgs& a, int pos) {
-    return a.temp_coef != 0.f ? 1.f + a.temp_coef * logf((float)floor(((double)pos + 1.0) / a.temp_every) + 1.f) : 1.f;
+    return a.temp_coef != 0.f ? 1.f + a.temp_coef * logf(floorf((float)(pos + 1) / a.temp_every) + 1.f) : 1.f;
 }
-// cap * tanh(s / cap) on the prompt path: below 1/8 the odd series x - x^3/3 + 2 x^5/15 (the next term is under 2.1e-7 of x), above it
-// 1 - 2 / (exp(2|x|) + 1), whose rounding errors stay near 1e-7 absolute
-__device__ __forceinline__ float sk_cap_fast(float s, float cap, float inv_cap) {
-    const float x = s * inv_cap, ax = fabsf(x), x2 = x * x;
-    const float series = fmaf(x2 * x, fmaf(x2, 2.f / 15.f, -1.f / 3.f), x);
-    const float big = copysignf(1.f - __fdividef(2.f, __expf(2.f * ax) + 1.f), x);
-    return cap * (ax < 0.125f ? series : big);
-}
+__device__ __forceinline__ float sk_exp2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+__device__ __forceinline__ float sk_rcp(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 }  // namespace
 
 constexpr int SK_MAXE = 8;       // key and value sizes <= 256
@@ -95,30 +91,40 @@ __global__ void __launch_bounds__(256) sink_attn_store_kernel(SinkAttnArgs a, Ra
 // ---------------------------------------------------------------- preparation with convolutions and whole-projection norms
 // grid (token groups, parts), NT threads. Part 0 = queries, 1 = keys, 2 = values, 3 = side columns: the parts share nothing, so a
 // decoded token is ready after the longest of them. A CTA takes up to TB neighbouring tokens of a segment: a thread walks its
-// channels, reads every projected row once for all TB outputs, and the rows wait in shared memory ([TB][channels], norms only) for
-// the sums of squares over all heads. Two grids:
+// channels, VEC neighbouring ones at a time, reads every projected row once for all TB outputs, and the rows wait in shared memory
+// ([TB][channels], norms only) for the sums of squares over all heads. Two grids:
 //   by tiles (prompts)          group = TB rows of a 64-row tile; the convolution state is moved on by a launch of its own afterwards
 //   by segments (few tokens)    group = a whole segment, TB tokens at a time; each thread then moves its channels' state on itself
-// Outputs are sums over the taps in tap order, the same in both.
-template <int TAPS>
-__device__ __forceinline__ float sk_conv(const SinkAttnArgs& a, const float* col, const float* w, int taps, int t, int i, const float* st, int C) {
-    const int n = TAPS > 0 ? TAPS : taps;
-    float acc = 0.f;
-#pragma unroll
-    for (int j = 0; j < n; j++) {
-        const int back = n - 1 - j;               // the input `back` tokens ago; before the step: the slot's last n - 1 inputs
-        const float v = i >= back ? col[(size_t)(t - back) * a.ldp] : st[(size_t)(n - 1 + i - back) * C];
-        acc = fmaf(w[j], v, acc);
-    }
-    return acc;
+// Outputs are sums over the taps in tap order, the same in both. TAPS: compiled number of taps, 1 = no convolution, 0 = any number.
+namespace {
+template <int VEC> struct SkVec { float v[VEC]; };
+template <int VEC>
+__device__ __forceinline__ SkVec<VEC> sk_vload(const float* p) {
+    SkVec<VEC> o;
+    if constexpr (VEC == 4) { const float4 f = *reinterpret_cast<const float4*>(p); o.v[0] = f.x; o.v[1] = f.y; o.v[2] = f.z; o.v[3] = f.w; }
+    else o.v[0] = *p;
+    return o;
 }
+template <int VEC>
+__device__ __forceinline__ void sk_vstore(float* p, const SkVec<VEC>& x) {
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(x.v[0], x.v[1], x.v[2], x.v[3]);
+    else *p = x.v[0];
+}
+template <int VEC>
+__device__ __forceinline__ void sk_vstore_bf16(__nv_bfloat16* p, const SkVec<VEC>& x) {
+    if constexpr (VEC == 4) {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(x.v[0], x.v[1]), b = __floats2bfloat162_rn(x.v[2], x.v[3]);
+        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+    } else *p = __float2bfloat16(x.v[0]);
+}
+}  // namespace
 
-template <int NT, int TB, int TAPS>
-__global__ void __launch_bounds__(NT) sink_attn_prepare_kernel(SinkAttnArgs a, RaggedDev r, int by_segment) {
+template <int NT, int TB, int TAPS, int VEC>
+__global__ void __launch_bounds__(NT, NT <= 256 ? 3 : 1) sink_attn_prepare_kernel(SinkAttnArgs a, RaggedDev r, int by_segment) {
     griddep_launch();
     griddep_wait();
-    extern __shared__ float pr_row[];                         // [TB][n]
-    __shared__ float red[TB][33];
+    extern __shared__ __align__(16) float pr_row[];           // [TB][n]
+    __shared__ float red[TB][32];
     const int part = blockIdx.y, nqd = a.H * a.d, nkd = a.G * a.d, nvd = a.G * a.dv, C = nqd + nkd + nvd;
     int seg, g0, g1;
     if (by_segment) {
@@ -131,53 +137,105 @@ __global__ void __launch_bounds__(NT) sink_attn_prepare_kernel(SinkAttnArgs a, R
         g1 = min(g0 + TB, r.seg_start[seg] + r.seg_len[seg]);
         if (g0 >= g1) return;
     }
-    const int start = r.seg_start[seg], slot = r.seg_slot[seg];
     if (part == 3) {
         for (int t = g0; t < g1; t++) {
             const float* row = a.proj + (size_t)t * a.ldp;
             const float gate = a.side_gate >= 0 ? sk_sigmoid(row[a.side_gate]) : 1.f;
-            for (int i = threadIdx.x; i < a.side_n; i += NT) a.out[(size_t)t * a.ld_out + a.side_col + i] = row[a.side_off + i] * gate;
+            const size_t to = (size_t)t * a.ld_out + a.side_col;
+            for (int i = threadIdx.x * VEC; i < a.side_n; i += NT * VEC) {
+                SkVec<VEC> x = sk_vload<VEC>(row + a.side_off + i);
+#pragma unroll
+                for (int e = 0; e < VEC; e++) x.v[e] *= gate;
+                if (a.out_bf16) sk_vstore_bf16<VEC>(a.out_bf16 + to + i, x);
+                else sk_vstore<VEC>(a.out + to + i, x);
+            }
         }
         return;
     }
+    const int start = r.seg_start[seg], slot = r.seg_slot[seg];
     const int n = part == 0 ? nqd : part == 1 ? nkd : nvd, off = part == 0 ? a.q_off : part == 1 ? a.k_off : a.v_off;
     const int ch0 = part == 0 ? 0 : part == 1 ? nqd : nqd + nkd, dd = part == 2 ? a.dv : a.d;
     const float* nw = part == 0 ? a.q_norm_w : part == 1 ? a.k_norm_w : nullptr;
     const int* table = a.block_tables[slot];
-    const float* state = a.conv_state ? a.conv_state + (size_t)slot * (a.taps - 1) * C + ch0 : nullptr;
+    const int taps = TAPS > 0 ? TAPS : a.conv_w ? a.taps : 1, hist = taps - 1;
+    const float* state = hist > 0 ? a.conv_state + (size_t)slot * hist * C + ch0 : nullptr;      // [hist][C], newest last
     for (int t0 = g0; t0 < g1; t0 += TB) {
         const int nt = min(TB, g1 - t0), i0 = t0 - start;
         size_t base[TB];                                      // of the token's row in the page (keys, values)
-        float mul[TB];
+        float mul[TB], ss[TB];
 #pragma unroll
         for (int u = 0; u < TB; u++) {
             const int t = min(t0 + u, g1 - 1), pos = r.tok_pos[t];
             base[u] = ((size_t)table[pos / a.block_tokens] * a.G * a.block_tokens + pos % a.block_tokens) * dd;
             mul[u] = part == 0 ? sk_temperature(a, pos) : 1.f;
+            ss[u] = 0.f;
         }
-        auto put = [&](int u, int c, float v) {
-            if (part == 0) { a.q_rot[(size_t)(t0 + u) * nqd + c] = v; return; }
-            const int g = c / dd;
-            sk_store(part == 1 ? a.k_pool : a.v_pool, a.cache_f32, base[u] + (size_t)g * a.block_tokens * dd + (c - g * dd), v);
+        // entry c of the part's row -> its place in the page, without the token's share
+        auto place = [&](int c) { const int g = part == 0 ? 0 : c / dd; return (size_t)g * a.block_tokens * dd + (c - g * dd); };
+        auto put = [&](int u, size_t at, SkVec<VEC> x, const SkVec<VEC>& w) {
+#pragma unroll
+            for (int e = 0; e < VEC; e++) x.v[e] *= mul[u] * w.v[e];
+            if (part == 0) { sk_vstore<VEC>(a.q_rot + (size_t)(t0 + u) * nqd + at, x); return; }
+            void* pool = part == 1 ? a.k_pool : a.v_pool;
+            if (a.cache_f32) sk_vstore<VEC>(reinterpret_cast<float*>(pool) + base[u] + at, x);
+            else sk_vstore_bf16<VEC>(reinterpret_cast<__nv_bfloat16*>(pool) + base[u] + at, x);
         };
-        float ss[TB];
+        SkVec<VEC> one;
 #pragma unroll
-        for (int u = 0; u < TB; u++) ss[u] = 0.f;
-        for (int c = threadIdx.x; c < n; c += NT) {
+        for (int e = 0; e < VEC; e++) one.v[e] = 1.f;
+        for (int c = threadIdx.x * VEC; c < n; c += NT * VEC) {
             const float* col = a.proj + off + c;
-            float w[TAPS > 0 ? TAPS : 1];
-            if (TAPS > 1)
+            SkVec<VEC> y[TB];
+            if constexpr (TAPS > 0) {
+                // the TB + TAPS - 1 inputs of the group, all in flight; before the step: the slot's last inputs
+                SkVec<VEC> in[TB + TAPS - 1];
 #pragma unroll
-                for (int j = 0; j < TAPS; j++) w[j] = a.conv_w[(size_t)(ch0 + c) * TAPS + j];
+                for (int k = 0; k < TB + TAPS - 1; k++) {
+                    const int i = i0 - (TAPS - 1) + k;        // token index within the segment
+                    in[k] = i >= 0 ? sk_vload<VEC>(col + (size_t)min(start + i, g1 - 1) * a.ldp) : sk_vload<VEC>(state + (size_t)(hist + i) * C + c);
+                }
+                if constexpr (TAPS == 1) {
+#pragma unroll
+                    for (int u = 0; u < TB; u++) y[u] = in[u];
+                } else {
+                    float w[VEC][TAPS];
+#pragma unroll
+                    for (int e = 0; e < VEC; e++)
+#pragma unroll
+                        for (int j = 0; j < TAPS; j++) w[e][j] = a.conv_w[(size_t)(ch0 + c + e) * TAPS + j];
+#pragma unroll
+                    for (int u = 0; u < TB; u++)
+#pragma unroll
+                        for (int e = 0; e < VEC; e++) {
+                            float acc = 0.f;
+#pragma unroll
+                            for (int j = 0; j < TAPS; j++) acc = fmaf(w[e][j], in[u + j].v[e], acc);
+                            y[u].v[e] = acc;
+                        }
+                }
+            } else {
+#pragma unroll
+                for (int u = 0; u < TB; u++) {
+#pragma unroll
+                    for (int e = 0; e < VEC; e++) y[u].v[e] = 0.f;
+                    if (u >= nt) continue;
+                    if (!a.conv_w) { y[u] = sk_vload<VEC>(col + (size_t)(t0 + u) * a.ldp); continue; }
+                    for (int j = 0; j < taps; j++) {
+                        const int i = i0 + u - hist + j;
+                        const SkVec<VEC> v = i >= 0 ? sk_vload<VEC>(col + (size_t)(start + i) * a.ldp) : sk_vload<VEC>(state + (size_t)(hist + i) * C + c);
+#pragma unroll
+                        for (int e = 0; e < VEC; e++) y[u].v[e] = fmaf(a.conv_w[(size_t)(ch0 + c + e) * taps + j], v.v[e], y[u].v[e]);
+                    }
+                }
+            }
+            const size_t at = nw ? 0 : place(c);
 #pragma unroll
             for (int u = 0; u < TB; u++) {
                 if (u >= nt) continue;
-                float v;
-                if (!a.conv_w) v = col[(size_t)(t0 + u) * a.ldp];
-                else if (TAPS > 1) v = sk_conv<TAPS>(a, col, w, TAPS, t0 + u, i0 + u, state + c, C);
-                else v = sk_conv<0>(a, col, a.conv_w + (size_t)(ch0 + c) * a.taps, a.taps, t0 + u, i0 + u, state + c, C);
-                if (nw) { pr_row[u * n + c] = v; ss[u] = fmaf(v, v, ss[u]); }
-                else put(u, c, v * mul[u]);
+                if (!nw) { put(u, at, y[u], one); continue; }
+                sk_vstore<VEC>(pr_row + u * n + c, y[u]);
+#pragma unroll
+                for (int e = 0; e < VEC; e++) ss[u] = fmaf(y[u].v[e], y[u].v[e], ss[u]);
             }
         }
         if (nw) {
@@ -195,37 +253,42 @@ __global__ void __launch_bounds__(NT) sink_attn_prepare_kernel(SinkAttnArgs a, R
                 for (int k = 0; k < NT / 32; k++) tot += red[u][k];
                 mul[u] *= 1.f / sqrtf(tot / (float)n + a.eps);
             }
-            for (int c = threadIdx.x; c < n; c += NT) {       // a thread reads back what it wrote itself
-                const float wv = nw[c];
+            for (int c = threadIdx.x * VEC; c < n; c += NT * VEC) {       // a thread reads back what it wrote itself
+                const SkVec<VEC> wv = sk_vload<VEC>(nw + c);
+                const size_t at = place(c);
 #pragma unroll
-                for (int u = 0; u < TB; u++) if (u < nt) put(u, c, pr_row[u * n + c] * mul[u] * wv);
+                for (int u = 0; u < TB; u++) if (u < nt) put(u, at, sk_vload<VEC>(pr_row + u * n + c), wv);
             }
         }
     }
-    if (by_segment && a.conv_w && a.taps > 1) {               // entry k of the new state is read at k + len > k of the old one before it is written
-        const int hist = a.taps - 1, len = g1 - g0;
-        for (int c = threadIdx.x; c < n; c += NT) {
-            float* st = a.conv_state + (size_t)slot * hist * C + ch0 + c;
+    if (by_segment && hist > 0) {                             // entry k of the new state is read at k + len > k of the old one before it is written
+        const int len = g1 - g0;
+        float* st = a.conv_state + (size_t)slot * hist * C + ch0;
+        for (int c = threadIdx.x * VEC; c < n; c += NT * VEC)
             for (int k = 0; k < hist; k++) {
                 const int src = len + k - hist;
-                st[(size_t)k * C] = src >= 0 ? a.proj[(size_t)(g0 + src) * a.ldp + off + c] : st[(size_t)(k + len) * C];
+                sk_vstore<VEC>(st + (size_t)k * C + c, src >= 0 ? sk_vload<VEC>(a.proj + (size_t)(g0 + src) * a.ldp + off + c)
+                                                                : sk_vload<VEC>(st + (size_t)(k + len) * C + c));
             }
-        }
     }
 }
 
+template <int NT, int TB, int TAPS, int VEC>
+static cudaError_t sink_attn_prepare_go(const SinkAttnArgs& a, const RaggedDev& r, dim3 grid, size_t smem, int by_segment, cudaStream_t s) {
+    static bool attr_done = false;
+    if (!attr_done) { cudaFuncSetAttribute(sink_attn_prepare_kernel<NT, TB, TAPS, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); attr_done = true; }
+    return launch_chain(sink_attn_prepare_kernel<NT, TB, TAPS, VEC>, grid, dim3(NT), smem, s, a, r, by_segment);
+}
 template <int NT, int TB>
 static cudaError_t sink_attn_prepare_pick(const SinkAttnArgs& a, const RaggedDev& r, dim3 grid, size_t smem, int by_segment, cudaStream_t s) {
-    static bool attr_done = false;
-    if (!attr_done) {
-        cudaFuncSetAttribute(sink_attn_prepare_kernel<NT, TB, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-        cudaFuncSetAttribute(sink_attn_prepare_kernel<NT, TB, 3>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-        cudaFuncSetAttribute(sink_attn_prepare_kernel<NT, TB, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-        attr_done = true;
-    }
-    if (a.conv_w && a.taps == 3) return launch_chain(sink_attn_prepare_kernel<NT, TB, 3>, grid, dim3(NT), smem, s, a, r, by_segment);
-    if (a.conv_w && a.taps == 4) return launch_chain(sink_attn_prepare_kernel<NT, TB, 4>, grid, dim3(NT), smem, s, a, r, by_segment);
-    return launch_chain(sink_attn_prepare_kernel<NT, TB, 0>, grid, dim3(NT), smem, s, a, r, by_segment);
+    // four channels at a time: rows, offsets and head sizes on 16-byte boundaries
+    const bool vec = ((a.ldp | a.q_off | a.k_off | a.v_off | a.d | a.dv) & 3) == 0 &&
+                     (a.side_n == 0 || ((a.side_off | a.side_n | a.side_col | a.ld_out) & 3) == 0);
+    const int taps = a.conv_w ? a.taps : 1;
+    if (vec && taps == 1 && !a.conv_w) return sink_attn_prepare_go<NT, TB, 1, 4>(a, r, grid, smem, by_segment, s);
+    if (vec && taps == 3) return sink_attn_prepare_go<NT, TB, 3, 4>(a, r, grid, smem, by_segment, s);
+    if (vec && taps == 4) return sink_attn_prepare_go<NT, TB, 4, 4>(a, r, grid, smem, by_segment, s);
+    return vec ? sink_attn_prepare_go<NT, TB, 0, 4>(a, r, grid, smem, by_segment, s) : sink_attn_prepare_go<NT, TB, 0, 1>(a, r, grid, smem, by_segment, s);
 }
 
 bool sink_attn_prepares(const SinkAttnArgs& a) { return a.q_norm_w || a.k_norm_w || a.conv_w || a.side_n > 0; }
@@ -411,6 +474,153 @@ __global__ void __launch_bounds__(128) sink_attn_talk_kernel(SinkAttnArgs a, int
     }
 }
 
+// The same attention for key and value sizes that are multiples of 8, without mixing across heads: 16-byte loads, LPK lanes per key
+// (8 entries each), 32 / LPK keys per warp and load, SK_U loads of keys and values in flight. Every group of LPK lanes keeps a running
+// maximum, sum and output of its own; they are merged once per CTA, in order. CL > 1 (few-token steps over many keys): the CL CTAs of
+// a cluster take CL equal ranges of the visible keys, leave (maximum, sum, output) in their shared memory, and each forms its share of
+// the output columns from all of them, in range order: one launch, nothing through global memory. grid (T, H, CL), 8 warps.
+constexpr int SK_U = 4;
+template <bool F32, int LPK, int CL>
+__device__ __forceinline__ void sink_attn_vec_body(const SinkAttnArgs& a, const RaggedDev& r) {
+    griddep_launch();
+    griddep_wait();
+    constexpr int S = 32 / LPK, PARTS = SK_WARPS * S, COLS = LPK * 8;
+    __shared__ float sm_o[PARTS][COLS], sm_m[PARTS], sm_l[PARTS], sm_f[PARTS];
+    __shared__ float cl_o[COLS], cl_ml[2];
+    const int t = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int sub = lane / LPK, c0 = (lane % LPK) * 8;
+    const int pos = r.tok_pos[t], d = a.d, dv = a.dv, g = h / (a.H / a.G);
+    const int* table = a.block_tables[r.seg_slot[r.tok_seg[t]]];
+    const float* q = a.q_rot + ((size_t)t * a.H + h) * d;
+    const float cap = a.softcap;
+    float qr[8], acc[8];
+#pragma unroll
+    for (int e = 0; e < 8; e++) { qr[e] = c0 < d ? q[c0 + e] * a.scale : 0.f; acc[e] = 0.f; }
+    float m_run = -INFINITY, l_run = 0.f;
+    int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0, hi = pos;
+    if (CL > 1) {                                             // this CTA's share of the visible keys
+        const int per = ((pos - lo + CL) / CL + PARTS - 1) / PARTS * PARTS;
+        lo += (int)blockIdx.z * per;
+        hi = min(pos, lo + per - 1);
+    }
+    auto load8 = [&](const void* pool, size_t i, bool on, float (&v)[8]) {
+        if constexpr (F32) {
+            const float4 x = on ? *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(pool) + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            const float4 y = on ? *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(pool) + i + 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+            v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
+        } else {
+            const uint4 x = on ? *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(pool) + i) : make_uint4(0, 0, 0, 0);
+            const uint32_t w[4] = {x.x, x.y, x.z, x.w};
+#pragma unroll
+            for (int e = 0; e < 4; e++) { v[2 * e] = __uint_as_float(w[e] << 16); v[2 * e + 1] = __uint_as_float(w[e] & 0xffff0000u); }
+        }
+    };
+    for (int b0 = lo; b0 <= hi; b0 += PARTS * SK_U) {
+        float kv[SK_U][8], vv[SK_U][8], sc[SK_U];
+        bool in[SK_U];
+#pragma unroll
+        for (int u = 0; u < SK_U; u++) {
+            const int j = b0 + u * PARTS + warp * S + sub;
+            in[u] = j <= hi;
+            const int jj = min(j, hi);                        // past the end: the last key again, its weight is dropped below
+            const size_t row = ((size_t)table[jj / a.block_tokens] * a.G + g) * a.block_tokens + jj % a.block_tokens;
+            load8(a.k_pool, row * d + c0, c0 < d, kv[u]);
+            load8(a.v_pool, row * dv + c0, c0 < dv, vv[u]);
+        }
+#pragma unroll
+        for (int u = 0; u < SK_U; u++) {
+            float dot = 0.f;
+#pragma unroll
+            for (int e = 0; e < 8; e++) dot = fmaf(qr[e], kv[u][e], dot);
+            sc[u] = dot;
+        }
+#pragma unroll
+        for (int o = LPK / 2; o > 0; o >>= 1)
+#pragma unroll
+            for (int u = 0; u < SK_U; u++) sc[u] += __shfl_xor_sync(0xffffffffu, sc[u], o);
+        if (cap > 0.f)
+#pragma unroll
+            for (int u = 0; u < SK_U; u++) sc[u] = cap * tanhf(sc[u] / cap);
+        float mx = m_run;
+#pragma unroll
+        for (int u = 0; u < SK_U; u++) if (in[u]) mx = fmaxf(mx, sc[u]);
+        const float ms = mx > -INFINITY ? mx : 0.f;           // no key of this group yet: every term is exp(-inf) = 0
+        const float corr = expf(m_run - ms);
+        l_run *= corr;
+#pragma unroll
+        for (int e = 0; e < 8; e++) acc[e] *= corr;
+#pragma unroll
+        for (int u = 0; u < SK_U; u++) {
+            const float p = in[u] ? expf(sc[u] - ms) : 0.f;
+            l_run += p;
+#pragma unroll
+            for (int e = 0; e < 8; e++) acc[e] = fmaf(p, vv[u][e], acc[e]);
+        }
+        m_run = mx;
+    }
+    const int part = warp * S + sub;
+#pragma unroll
+    for (int e = 0; e < 8; e++) sm_o[part][c0 + e] = acc[e];
+    if (lane % LPK == 0) { sm_m[part] = m_run; sm_l[part] = l_run; }
+    __syncthreads();
+    const float sink = a.sink && CL == 1 ? a.sink[h] : -INFINITY;
+    if (warp == 0) {
+        const float mk = lane < PARTS ? sm_m[lane] : -INFINITY;
+        const float m = fmaxf(warp_max(mk), sink);
+        const float f = mk > -INFINITY ? expf(mk - m) : 0.f;
+        const float l = warp_sum(lane < PARTS ? sm_l[lane] * f : 0.f) + (sink > -INFINITY ? expf(sink - m) : 0.f);
+        if (lane < PARTS) sm_f[lane] = f;
+        if (lane == 0) { cl_ml[0] = m; cl_ml[1] = l; }
+    }
+    __syncthreads();
+    const float inv = CL > 1 ? 1.f : 1.f / cl_ml[1];
+    for (int i = threadIdx.x; i < dv; i += blockDim.x) {
+        float o = 0.f;
+#pragma unroll
+        for (int k = 0; k < PARTS; k++) o = fmaf(sm_o[k][i], sm_f[k], o);
+        if (CL > 1) cl_o[i] = o;
+        else a.out[(size_t)t * a.ld_out + (size_t)h * dv + i] = o * inv * sk_gate(a, t, h, i);
+    }
+    if constexpr (CL > 1) {
+        namespace cg = cooperative_groups;
+        cg::cluster_group cluster = cg::this_cluster();
+        cluster.sync();
+        const float snk = a.sink ? a.sink[h] : -INFINITY;
+        const int per = (dv + CL - 1) / CL, i = (int)blockIdx.z * per + (int)threadIdx.x;
+        if ((int)threadIdx.x < per && i < dv) {
+            float m = snk, mr[CL], o = 0.f;
+#pragma unroll
+            for (int k = 0; k < CL; k++) { mr[k] = cluster.map_shared_rank(cl_ml, k)[0]; m = fmaxf(m, mr[k]); }
+            float l = snk > -INFINITY ? expf(snk - m) : 0.f;
+#pragma unroll
+            for (int k = 0; k < CL; k++) {
+                const float f = mr[k] > -INFINITY ? expf(mr[k] - m) : 0.f;
+                l = fmaf(cluster.map_shared_rank(cl_ml, k)[1], f, l);
+                o = fmaf(cluster.map_shared_rank(cl_o, k)[i], f, o);
+            }
+            a.out[(size_t)t * a.ld_out + (size_t)h * dv + i] = o / l * sk_gate(a, t, h, i);
+        }
+        cluster.sync();                                       // nobody leaves while others read its shared memory
+    }
+}
+template <bool F32, int LPK>
+__global__ void __launch_bounds__(SK_WARPS * 32) sink_attn_vec_kernel(SinkAttnArgs a, RaggedDev r) { sink_attn_vec_body<F32, LPK, 1>(a, r); }
+constexpr int SK_CLUSTER = 8;
+template <bool F32, int LPK>
+__global__ void __cluster_dims__(1, 1, SK_CLUSTER) __launch_bounds__(SK_WARPS * 32) sink_attn_cluster_kernel(SinkAttnArgs a, RaggedDev r) {
+    sink_attn_vec_body<F32, LPK, SK_CLUSTER>(a, r);
+}
+template <bool F32>
+static cudaError_t sink_attn_vec_launch(const SinkAttnArgs& a, const RaggedDev& r, cudaStream_t s) {
+    const int n = std::max(a.d, a.dv);
+    // which form runs depends on the step's shape and the most keys a query can see, never on the positions: a captured step can be replayed
+    const bool cl = r.T <= SK_FEW_TOKENS && a.max_keys > 256;
+    const dim3 grid(r.T, a.H, cl ? SK_CLUSTER : 1), block(SK_WARPS * 32);
+    if (n <= 64) return launch_chain(cl ? sink_attn_cluster_kernel<F32, 8> : sink_attn_vec_kernel<F32, 8>, grid, block, 0, s, a, r);
+    if (n <= 128) return launch_chain(cl ? sink_attn_cluster_kernel<F32, 16> : sink_attn_vec_kernel<F32, 16>, grid, block, 0, s, a, r);
+    return launch_chain(cl ? sink_attn_cluster_kernel<F32, 32> : sink_attn_vec_kernel<F32, 32>, grid, block, 0, s, a, r);
+}
+
 // Tensor-core prompt attention (bf16 pages, key and value sizes multiples of 16 up to 128): a CTA takes one tile of up to 64
 // consecutive queries of a segment, one query head and one value head; 4 warps x 16 query rows; keys in blocks of 64 from the block
 // that holds the oldest key of the tile's first query to the block of its last query, staged in shared memory once for all 64
@@ -461,11 +671,16 @@ __global__ void __launch_bounds__(128) sink_attn_mma_kernel(SinkAttnArgs a, Ragg
     const int vg = a.talk ? (int)(blockIdx.y % Gv) : g;
     const __nv_bfloat16* kp = reinterpret_cast<const __nv_bfloat16*>(a.k_pool);
     const __nv_bfloat16* vp = reinterpret_cast<const __nv_bfloat16*>(a.v_pool);
+    // scores live in the log2 domain (exp2 below). Capped: cap tanh(s / cap) = cap - 2 cap / (exp(2 s / cap) + 1), the exponential's
+    // factor folded into the query as well; its rounding error is about 1e-7 of the cap
+    constexpr float LOG2E = 1.4426950408889634f;
+    const float q_mul = CAP ? a.scale * (2.f * LOG2E) / a.softcap : a.scale * LOG2E;
+    [[maybe_unused]] const float cap2 = CAP ? a.softcap * LOG2E : 0.f;
     for (int i = threadIdx.x; i < SKM_Q * (d / 2); i += blockDim.x) {
         const int rr = i / (d / 2), c = (i % (d / 2)) * 2;
         float2 v = make_float2(0.f, 0.f);
         if (rr < nq) v = *reinterpret_cast<const float2*>(a.q_rot + ((size_t)(row0 + rr) * a.H + h) * d + c);
-        v.x *= a.scale; v.y *= a.scale;
+        v.x *= q_mul; v.y *= q_mul;
         const __nv_bfloat162 hi = __floats2bfloat162_rn(v.x, v.y);
         *reinterpret_cast<__nv_bfloat162*>(Qs + rr * LD + c) = hi;
         *reinterpret_cast<__nv_bfloat162*>(Ql + rr * LD + c) = __floats2bfloat162_rn(v.x - __low2float(hi), v.y - __high2float(hi));
@@ -479,32 +694,37 @@ __global__ void __launch_bounds__(128) sink_attn_mma_kernel(SinkAttnArgs a, Ragg
     const int qrow[2] = {warp * 16 + gq, warp * 16 + gq + 8};
     int qlo[2];                                    // oldest visible key of the lane's two query rows
     float m_run[2], l_run[2];
-    const float sink = a.sink ? a.sink[h] : -INFINITY;
-    [[maybe_unused]] const float inv_cap = CAP ? 1.f / a.softcap : 0.f;
+    const float sink = a.sink ? a.sink[h] * LOG2E : -INFINITY;
 #pragma unroll
     for (int q2 = 0; q2 < 2; q2++) {
         const int i = p0 + qrow[q2];
         qlo[q2] = a.window > 0 ? max(0, i - a.window + 1) : 0;
         m_run[q2] = sink; l_run[q2] = 0.f;         // the running maximum starts at the sink; its term joins the sum at the end
     }
-    for (int kb = b0; kb <= b1; kb++) {
-        const int j0 = kb * SKM_K;
-        __syncthreads();                      // everybody is done with the previous block's K and V (and Q is written)
-        for (int i = threadIdx.x; i < SKM_K * (d / 8); i += blockDim.x) {
-            const int rr = i / (d / 8), c = (i % (d / 8)) * 8;
-            const int j = j0 + rr, jj = min(j, p_last);
-            const size_t base = (((size_t)table[jj / a.block_tokens] * a.G + g) * a.block_tokens + jj % a.block_tokens) * d + c;
-            sk_cp_async_16z(Ks + rr * LD + c, kp + base, j <= p_last ? 16 : 0);
-        }
-        for (int i = threadIdx.x; i < SKM_K * (dv / 8); i += blockDim.x) {
-            const int rr = i / (dv / 8), c = (i % (dv / 8)) * 8;
-            const int j = j0 + rr, jj = min(j, p_last);
-            const size_t base = (((size_t)table[jj / a.block_tokens] * a.G + vg) * a.block_tokens + jj % a.block_tokens) * dv + c;
-            sk_cp_async_16z(Vs + rr * LDV + c, vp + base, j <= p_last ? 16 : 0);
+    // the next block's keys arrive while this block's weights meet the values, its values while the next scores are formed
+    // (the thread's chunks of 16 bytes advance through the block without divisions; pages that hold whole blocks are looked up once)
+    const bool whole = a.block_tokens % SKM_K == 0;
+    auto load_rows = [&](const __nv_bfloat16* pool, int head, int n, int ld, __nv_bfloat16* dst, int kb) {
+        const int per = n / 8, j0 = kb * SKM_K, last = p_last - j0;     // rows past `last` are zero
+        int rr = threadIdx.x / per, c = threadIdx.x - rr * per;
+        const int drr = 128 / per, dc = 128 - drr * per;
+        const __nv_bfloat16* block = whole ? pool + (((size_t)table[j0 / a.block_tokens] * a.G + head) * a.block_tokens + j0 % a.block_tokens) * n : nullptr;
+        while (rr < SKM_K) {
+            const int row = min(rr, last);
+            const __nv_bfloat16* src = whole ? block + row * n
+                                             : pool + (((size_t)table[(j0 + row) / a.block_tokens] * a.G + head) * a.block_tokens + (j0 + row) % a.block_tokens) * n;
+            sk_cp_async_16z(dst + rr * ld + c * 8, src + c * 8, rr <= last ? 16 : 0);
+            rr += drr; c += dc;
+            if (c >= per) { c -= per; rr++; }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
-        asm volatile("cp.async.wait_group 0;" ::: "memory");
-        __syncthreads();
+    };
+    load_rows(kp, g, d, LD, Ks, b0);
+    load_rows(vp, vg, dv, LDV, Vs, b0);
+    for (int kb = b0; kb <= b1; kb++) {
+        const int j0 = kb * SKM_K;
+        asm volatile("cp.async.wait_group 1;" ::: "memory");          // this block's keys (its values may still be on their way)
+        __syncthreads();                                                // ... everybody's share of them (and Q is written)
         float sacc[SKM_K / 8][4];
 #pragma unroll
         for (int ni = 0; ni < SKM_K / 8; ni++) sacc[ni][0] = sacc[ni][1] = sacc[ni][2] = sacc[ni][3] = 0.f;
@@ -525,32 +745,46 @@ __global__ void __launch_bounds__(128) sink_attn_mma_kernel(SinkAttnArgs a, Ragg
                 }
             }
         }
+        __syncthreads();                                                // everybody is done with the keys
+        if (kb < b1) load_rows(kp, g, d, LD, Ks, kb + 1);
+        else asm volatile("cp.async.commit_group;" ::: "memory");      // keep the count of groups
         // mask, running maximum per query row (a row lives in the four lanes of a quad), probabilities
         float mx[2] = {m_run[0], m_run[1]};
+        if constexpr (CAP)
+#pragma unroll
+            for (int ni = 0; ni < SKM_K / 8; ni++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) sacc[ni][e] = fmaf(-2.f * cap2, sk_rcp(sk_exp2(sacc[ni][e]) + 1.f), cap2);
+        // the warp's rows all see the whole block: from its last key on, and not beyond the oldest key of its last row
+        const int w_first = p0 + warp * 16, w_last = w_first + 15;
+        const bool all = warp * 16 + 15 < nq && j0 + SKM_K - 1 <= w_first && (a.window <= 0 || j0 > w_last - a.window);
+        if (!all)
+#pragma unroll
+            for (int ni = 0; ni < SKM_K / 8; ni++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const int rr = qrow[e >> 1], i = p0 + rr, j = j0 + ni * 8 + 2 * tq + (e & 1);
+                    const bool vis = rr < nq && j <= i && j >= qlo[e >> 1];
+                    sacc[ni][e] = vis ? sacc[ni][e] : -INFINITY;
+                }
 #pragma unroll
         for (int ni = 0; ni < SKM_K / 8; ni++)
 #pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int rr = qrow[e >> 1], i = p0 + rr, j = j0 + ni * 8 + 2 * tq + (e & 1);
-                const bool vis = rr < nq && j <= i && j >= qlo[e >> 1];
-                if constexpr (CAP) sacc[ni][e] = sk_cap_fast(sacc[ni][e], a.softcap, inv_cap);
-                sacc[ni][e] = vis ? sacc[ni][e] : -INFINITY;
-                mx[e >> 1] = fmaxf(mx[e >> 1], sacc[ni][e]);
-            }
+            for (int e = 0; e < 4; e++) mx[e >> 1] = fmaxf(mx[e >> 1], sacc[ni][e]);
         float corr[2], msafe[2], rs[2] = {0.f, 0.f};
 #pragma unroll
         for (int q2 = 0; q2 < 2; q2++) {
             mx[q2] = fmaxf(mx[q2], __shfl_xor_sync(0xffffffffu, mx[q2], 1));
             mx[q2] = fmaxf(mx[q2], __shfl_xor_sync(0xffffffffu, mx[q2], 2));
             msafe[q2] = mx[q2] > -INFINITY ? mx[q2] : 0.f;             // nothing visible yet and no sink: every term is exp(-inf) = 0
-            corr[q2] = __expf(m_run[q2] - msafe[q2]);
+            corr[q2] = sk_exp2(m_run[q2] - msafe[q2]);
             m_run[q2] = mx[q2];
         }
 #pragma unroll
         for (int ni = 0; ni < SKM_K / 8; ni++)
 #pragma unroll
             for (int e = 0; e < 4; e++) {
-                const float p = __expf(sacc[ni][e] - msafe[e >> 1]);
+                const float p = sk_exp2(sacc[ni][e] - msafe[e >> 1]);
                 sacc[ni][e] = p;
                 rs[e >> 1] += p;
             }
@@ -562,6 +796,8 @@ __global__ void __launch_bounds__(128) sink_attn_mma_kernel(SinkAttnArgs a, Ragg
         }
 #pragma unroll
         for (int i = 0; i < DVMAX / 8; i++) { o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1]; }
+        asm volatile("cp.async.wait_group 1;" ::: "memory");          // this block's values
+        __syncthreads();
 #pragma unroll
         for (int kc = 0; kc < SKM_K / 16; kc++) {
             uint32_t pf[4], pl[4];
@@ -581,11 +817,13 @@ __global__ void __launch_bounds__(128) sink_attn_mma_kernel(SinkAttnArgs a, Ragg
                 }
             }
         }
+        __syncthreads();                                                // everybody is done with the values
+        if (kb < b1) load_rows(vp, vg, dv, LDV, Vs, kb + 1);
     }
     float inv[2];
 #pragma unroll
     for (int q2 = 0; q2 < 2; q2++) {
-        const float l = l_run[q2] + (a.sink ? __expf(sink - m_run[q2]) : 0.f);
+        const float l = l_run[q2] + (a.sink ? sk_exp2(sink - m_run[q2]) : 0.f);
         inv[q2] = l > 0.f ? 1.f / l : 0.f;
     }
 #pragma unroll
@@ -596,6 +834,13 @@ __global__ void __launch_bounds__(128) sink_attn_mma_kernel(SinkAttnArgs a, Ragg
             if (rr >= nq || c >= dv) continue;
             const float v = o[i][e] * inv[e >> 1];
             const int t = row0 + rr;
+            if (a.out_bf16) {                  // two neighbouring columns of a row (dv is even)
+                if (e & 1) continue;
+                const float v2 = o[i][e + 1] * inv[e >> 1];
+                *reinterpret_cast<__nv_bfloat162*>(a.out_bf16 + (size_t)t * a.ld_out + (size_t)h * dv + c) =
+                    __floats2bfloat162_rn(v * sk_gate(a, t, h, c), v2 * sk_gate(a, t, h, c + 1));
+                continue;
+            }
             if (a.talk) a.cross[(((size_t)t * a.H + h) * a.G + vg) * dv + c] = v;
             else a.out[(size_t)t * a.ld_out + (size_t)h * dv + c] = v * sk_gate(a, t, h, c);
         }
@@ -893,17 +1138,24 @@ static cudaError_t sink_attn_mma_sizes(const SinkAttnArgs& a, const RaggedDev& r
     return a.dv <= 64 ? sink_attn_mma_pick<128, 64, CAP>(a, r, s) : sink_attn_mma_pick<128, 128, CAP>(a, r, s);
 }
 
+bool sink_attn_on_tensor_cores(const SinkAttnArgs& a, int T) {
+    static const bool no_mma = getenv("B2_NO_ATTN_MMA") != nullptr;        // tuning aid: scalar attention for prompts too
+    return !no_mma && !a.cache_f32 && T > SK_FEW_TOKENS && a.d % 16 == 0 && a.dv % 16 == 0 && a.d <= 128 && a.dv <= 128;
+}
+
 cudaError_t sink_attn_launch(const SinkAttnArgs& a, const RaggedDev& r, cudaStream_t s) {
     if (a.d > SK_MAXE * 32 || a.dv > SK_MAXE * 32 || a.H % a.G || (a.talk && a.softcap > 0.f)) return cudaErrorInvalidValue;
-    static const bool no_mma = getenv("B2_NO_ATTN_MMA") != nullptr;        // tuning aid: scalar attention for prompts too
     const int Gv = a.talk ? a.G : 1;
     cudaError_t e;
-    if (!no_mma && !a.cache_f32 && r.T > SK_FEW_TOKENS && a.d % 16 == 0 && a.dv % 16 == 0 && a.d <= 128 && a.dv <= 128) {
+    if (a.out_bf16 && !sink_attn_on_tensor_cores(a, r.T)) return cudaErrorInvalidValue;
+    if (sink_attn_on_tensor_cores(a, r.T)) {
         static const bool no_mixed = getenv("B2_NO_ATTN_MIXED") != nullptr;    // tuning aid: one weighted sum per (query head, value head) pair
         // with one or two key/value heads the separate sums cost no more than the second score pass and the scratch traffic
         // (measured at 8 heads over 2: 0.84 against 1.08 ms for four layers and 2048 tokens)
         if (a.talk && a.G >= 3 && !no_mixed && sink_attn_mixed_launch(a, r, s, e)) return e;
         e = a.softcap > 0.f ? sink_attn_mma_sizes<true>(a, r, s) : sink_attn_mma_sizes<false>(a, r, s);
+    } else if (!a.talk && a.d % 8 == 0 && a.dv % 8 == 0) {
+        return a.cache_f32 ? sink_attn_vec_launch<true>(a, r, s) : sink_attn_vec_launch<false>(a, r, s);
     } else {
         // few tokens: enough key ranges to fill the GPU; the count depends on the step's shape and the window only, never on the
         // positions, so that a captured step can be replayed
