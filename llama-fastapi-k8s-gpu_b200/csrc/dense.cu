@@ -38,23 +38,23 @@ struct DenseDev {
 // The rows [t0, t1) this CTA computes and the operands they use. false: nothing to do.
 template <typename TW>
 __device__ __forceinline__ bool dense_tile(const DenseDev& a, int rows_per_cta, const float*& x, const TW*& w, float*& y, const float*& aux,
-                                           int& t0, int& t1) {
+                                           int& t0, int& t1, int by, int bz) {
     x = a.x; w = reinterpret_cast<const TW*>(a.w); y = a.y; aux = a.aux;
     if (a.grouped == 0) {
-        const long b = blockIdx.z;
+        const long b = bz;
         x += b * a.x_bs; w += b * a.w_bs; y += b * a.y_bs;
         if (aux) aux += b * a.aux_bs;
-        t0 = blockIdx.y * rows_per_cta; t1 = a.T;
+        t0 = by * rows_per_cta; t1 = a.T;
         return t0 < t1;
     }
     if (a.grouped == 1) {
-        const int p = blockIdx.y, g = a.g.group[p];
+        const int p = by, g = a.g.group[p];
         if (g < 0 || g >= a.g.n_groups) return false;
         w += (long)g * a.g.w_stride;
         t0 = p; t1 = p + 1;
         return true;
     }
-    const int tile = blockIdx.y;
+    const int tile = by;
     if (tile >= *a.g.n_tiles) return false;
     w += (long)a.g.tile_group[tile] * a.g.w_stride;
     t0 = a.g.tile_row0[tile]; t1 = t0 + a.g.tile_rows[tile];
@@ -119,16 +119,14 @@ __device__ __forceinline__ void epi_store2(const DenseDev& a, float* y, const fl
 // over k in an order that depends on K alone.
 constexpr int ROWS_MAX_T = 8;
 template <typename TW, int TT, int R>
-__global__ void __launch_bounds__(256) dense_rows_kernel(DenseDev a) {
-    griddep_launch();
-    griddep_wait();
+__device__ __forceinline__ void dense_rows_cta(const DenseDev& a, int bx, int by, int bz) {
     constexpr int U = 4 / R;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int N = a.N, K = a.K, ldx = a.ldx;
-    const int n0 = (blockIdx.x * 8 + warp) * R;
+    const int n0 = (bx * 8 + warp) * R;
     if (n0 >= N) return;
     const float* x; const TW* w; float* y; const float* aux; int t0, t1;
-    if (!dense_tile<TW>(a, ROWS_MAX_T, x, w, y, aux, t0, t1)) return;
+    if (!dense_tile<TW>(a, ROWS_MAX_T, x, w, y, aux, t0, t1, by, bz)) return;
     const int T = a.grouped ? 1 : a.T;
     const float* rs = a.g.row_scale;
     if (a.grouped) { x += (size_t)x_row(a, t0) * ldx; y += (size_t)t0 * a.ldy; if (aux) aux += (size_t)t0 * a.ldaux; if (rs) rs += t0; }
@@ -211,6 +209,20 @@ __global__ void __launch_bounds__(256) dense_rows_kernel(DenseDev a) {
         }
     }
 }
+template <typename TW, int TT, int R>
+__global__ void __launch_bounds__(256) dense_rows_kernel(DenseDev a) {
+    griddep_launch();
+    griddep_wait();
+    dense_rows_cta<TW, TT, R>(a, blockIdx.x, blockIdx.y, blockIdx.z);
+}
+// two independent products in one launch: the CTAs of a, then those of b (grouped pairs, `nb` CTAs each)
+template <typename TW, int TT, int R>
+__global__ void __launch_bounds__(256) dense_rows_pair_kernel(DenseDev a, DenseDev b, int na, int nb) {
+    griddep_launch();
+    griddep_wait();
+    if ((int)blockIdx.x < na) dense_rows_cta<TW, TT, R>(a, blockIdx.x, 0, 0);
+    else dense_rows_cta<TW, 1, 1>(b, (blockIdx.x - na) % nb, (blockIdx.x - na) / nb, 0);
+}
 
 template <typename TW>
 static cudaError_t launch_rows(const DenseDev& d, int batch, cudaStream_t s) {
@@ -235,7 +247,7 @@ __global__ void __launch_bounds__(256) dense_fma_kernel(DenseDev a) {
     __shared__ float xs[BK][BM + 4];
     __shared__ float ws[BK][BN + 4];
     const float* x; const TW* w; float* y; const float* aux; int t0, T;
-    if (!dense_tile<TW>(a, BM, x, w, y, aux, t0, T)) return;
+    if (!dense_tile<TW>(a, BM, x, w, y, aux, t0, T, blockIdx.y, blockIdx.z)) return;
     const int N = a.N, K = a.K, ldx = a.ldx;
     const int n0 = blockIdx.x * BN;
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;      // thread tile: rows ty*4.., cols tx*4..
@@ -285,7 +297,7 @@ __global__ void __launch_bounds__(128) dense_mma_kernel(DenseDev a) {
     __shared__ __align__(16) __nv_bfloat16 xs[BM][LD];
     __shared__ __align__(16) __nv_bfloat16 ws[BN][LD];
     const float* x; const __nv_bfloat16* w; float* y; const float* aux; int t0, T;
-    if (!dense_tile<__nv_bfloat16>(a, BM, x, w, y, aux, t0, T)) return;
+    if (!dense_tile<__nv_bfloat16>(a, BM, x, w, y, aux, t0, T, blockIdx.y, blockIdx.z)) return;
     const int N = a.N, K = a.K, ldx = a.ldx;
     const int n0 = blockIdx.x * BN;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -391,7 +403,7 @@ __global__ void __launch_bounds__(256, 2) dense_mma_big_kernel(const __nv_bfloat
     __nv_bfloat16* As = reinterpret_cast<__nv_bfloat16*>(big_smem);                       // [stage][BM][LD]
     __nv_bfloat16* Bs = As + BIG_STAGES * BIG_BM * BIG_LD;                                  // [stage][BN][LD]
     const float* x; const __nv_bfloat16* w; float* y; const float* aux; int t0, T;
-    if (!dense_tile<__nv_bfloat16>(a, BIG_BM, x, w, y, aux, t0, T)) return;
+    if (!dense_tile<__nv_bfloat16>(a, BIG_BM, x, w, y, aux, t0, T, blockIdx.y, blockIdx.z)) return;
     const int N = a.N, K = a.K;
     const int n0 = blockIdx.x * BIG_BN;
     // the rounded copy holds the input rows as [row][ldxb] (grouped: gathered here; batched: batch b starts at column b * x_bs)
@@ -471,16 +483,41 @@ bool dense_takes_rounded(const DenseArgs& a) {
     return ok && (a.groups ? tiled && a.groups->tile_max == BIG_BM : a.T >= 64);
 }
 
+static DenseDev dense_dev(const DenseArgs& a) {
+    DenseDev d = {};
+    d.x = a.x; d.ldx = a.ldx; d.w = a.w; d.bias = a.bias; d.y = a.y; d.ldy = a.ldy; d.T = a.T; d.N = a.N; d.K = a.K; d.epi = a.epi;
+    d.n_act = a.n_act; d.n_act_end = a.n_act_end; d.yb = a.y_rounded; d.scale = a.scale; d.p0 = a.p0; d.p1 = a.p1;
+    d.aux = a.aux; d.ldaux = a.ldaux; d.aux_ns = a.aux_one ? 0 : 1; d.x_bs = a.x_bs; d.w_bs = a.w_bs; d.y_bs = a.y_bs; d.aux_bs = a.aux_bs;
+    if (a.groups) { d.g = *a.groups; d.grouped = a.groups->tile_group ? 2 : 1; }
+    return d;
+}
+
+static bool glu_epi(int epi) { return epi == EPI_GLU_SILU || epi == EPI_GLU_GELU || epi == EPI_GLU_CLAMP; }
+bool dense_pairs(const DenseArgs& a, const DenseArgs& b) {
+    return !a.groups && a.batch == 1 && a.T >= 1 && a.T <= ROWS_MAX_T && b.groups && !b.groups->tile_group && a.w_type == b.w_type &&
+           !glu_epi(a.epi) && !glu_epi(b.epi) && !a.x_rounded && !a.y_rounded && !b.x_rounded && !b.y_rounded;
+}
+template <typename TW>
+static cudaError_t launch_rows_pair(const DenseDev& a, const DenseDev& b, cudaStream_t s) {
+    const int per = a.T == 1 ? 8 : a.T == 2 ? 16 : 32, na = (a.N + per - 1) / per, nb = (b.N + 7) / 8;      // rows per CTA as in launch_rows
+    const dim3 grid(na + nb * b.T), block(256);
+    if (a.T == 1) return launch_chain(dense_rows_pair_kernel<TW, 1, 1>, grid, block, 0, s, a, b, na, nb);
+    if (a.T == 2) return launch_chain(dense_rows_pair_kernel<TW, 2, 2>, grid, block, 0, s, a, b, na, nb);
+    if (a.T <= 4) return launch_chain(dense_rows_pair_kernel<TW, 4, 4>, grid, block, 0, s, a, b, na, nb);
+    return launch_chain(dense_rows_pair_kernel<TW, 8, 4>, grid, block, 0, s, a, b, na, nb);
+}
+cudaError_t dense_pair_launch(const DenseArgs& a, const DenseArgs& b, cudaStream_t s) {
+    if (!dense_pairs(a, b) || a.N <= 0 || a.K <= 0 || b.T <= 0 || b.N <= 0 || b.K <= 0) return cudaErrorInvalidValue;
+    return a.w_type == T_BF16 ? launch_rows_pair<__nv_bfloat16>(dense_dev(a), dense_dev(b), s) : launch_rows_pair<float>(dense_dev(a), dense_dev(b), s);
+}
+
 cudaError_t dense_launch(const DenseArgs& a, cudaStream_t s) {
     if (a.T <= 0 || a.N <= 0 || a.K <= 0 || a.batch <= 0) return cudaErrorInvalidValue;
     if (a.w_type != T_BF16 && a.w_type != T_F32) return cudaErrorInvalidValue;
-    if ((a.epi == EPI_GLU_SILU || a.epi == EPI_GLU_GELU || a.epi == EPI_GLU_CLAMP) && a.N % 2) return cudaErrorInvalidValue;
+    if (glu_epi(a.epi) && a.N % 2) return cudaErrorInvalidValue;
     if (a.groups && a.batch != 1) return cudaErrorInvalidValue;
     const bool wb = a.w_type == T_BF16;
-    DenseDev d = {};
-    d.x = a.x; d.ldx = a.ldx; d.w = a.w; d.bias = a.bias; d.y = a.y; d.ldy = a.ldy; d.T = a.T; d.N = a.N; d.K = a.K; d.epi = a.epi;
-    d.n_act = a.n_act; d.n_act_end = a.n_act_end; d.yb = a.y_rounded; d.scale = a.scale; d.p0 = a.p0; d.p1 = a.p1; d.aux = a.aux; d.ldaux = a.ldaux; d.aux_ns = a.aux_one ? 0 : 1; d.x_bs = a.x_bs; d.w_bs = a.w_bs; d.y_bs = a.y_bs; d.aux_bs = a.aux_bs;
-    if (a.groups) { d.g = *a.groups; d.grouped = a.groups->tile_group ? 2 : 1; }
+    const DenseDev d = dense_dev(a);
     if (d.grouped == 1 || (!d.grouped && a.T <= ROWS_MAX_T)) return wb ? launch_rows<__nv_bfloat16>(d, a.batch, s) : launch_rows<float>(d, a.batch, s);
     // few output columns in 32-bit (router scores): the tiled kernel would run a handful of CTAs over the whole K; the
     // few-token kernel over chunks of 8 rows keeps every SM busy and streams the small matrix from L2

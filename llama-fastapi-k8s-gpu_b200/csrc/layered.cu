@@ -20,6 +20,7 @@
 #include <string.h>
 
 #include <algorithm>
+#include <utility>
 
 namespace b2 {
 
@@ -103,6 +104,8 @@ struct LayeredModel {
     // blocks behind one norm: what a producer leaves already rounded for the large products: the normed row, the mixer's output row;
     // experts' activations (every family)
     __nv_bfloat16 *hn_b = nullptr, *mix_b = nullptr, *moe_hb = nullptr;
+    // few-token steps: an expert product that the mixer's next product takes along in its launch (cleared when it has)
+    const DenseArgs* rider = nullptr;
     const __nv_bfloat16* hn_rounded = nullptr;      // hn_b when the step's boundary kernels fill it
     std::unordered_map<std::string, StepGraph> graphs;     // replayable small steps, by shape (b2_step)
     bool graphs_on = true;
@@ -965,15 +968,25 @@ struct StepProfiler {                 // events around launches of one kind, onl
 };
 }  // namespace
 
-static int dense(b2_engine* e, LayeredModel* m, const DenseW& w, const float* x, int ldx, float* y, int ldy, int T,
-                 const float* bias = nullptr, int epi = EPI_NONE, int kind = 1, DenseArgs* more = nullptr) {
-    StepProfiler sp(m, e->stream, kind);
+static DenseArgs dense_args(const LayeredModel* m, const DenseW& w, const float* x, int ldx, float* y, int ldy, int T, const float* bias, int epi,
+                            const DenseArgs* more) {
     DenseArgs a = more ? *more : DenseArgs{};
     a.x = x; a.ldx = ldx; a.w = w.w; a.w_type = w.type; a.bias = bias; a.y = y; a.ldy = ldy; a.T = T; a.N = w.N; a.K = w.K;
     a.epi = epi; a.exact = m->exact || (more && more->exact); a.xb = m->xb;
-    CK(dense_launch(a, e->stream));
+    return a;
+}
+static int dense_run(b2_engine* e, LayeredModel* m, const DenseArgs& a, int kind) {
+    StepProfiler sp(m, e->stream, kind);
+    if (m->rider && dense_pairs(a, *m->rider)) {
+        CK(dense_pair_launch(a, *m->rider, e->stream));
+        m->rider = nullptr;
+    } else CK(dense_launch(a, e->stream));
     e->launches++;
     return B2_OK;
+}
+static int dense(b2_engine* e, LayeredModel* m, const DenseW& w, const float* x, int ldx, float* y, int ldy, int T,
+                 const float* bias = nullptr, int epi = EPI_NONE, int kind = 1, const DenseArgs* more = nullptr) {
+    return dense_run(e, m, dense_args(m, w, x, ldx, y, ldy, T, bias, epi, more), kind);
 }
 
 // a plain product of T rows with these weights takes inputs that are rounded already
@@ -1210,7 +1223,8 @@ static int mix_chunk_linear(b2_engine* e, LayeredModel* m, LyLayer& L, const Rag
 
 // softmax attention with a sink, alone (output in m->oL) or beside the head-decay delta rule (attention in m->oL, delta rule in
 // m->oR; the caller norms and averages them)
-static int mix_sink(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in) {
+// (riders[0 / 1]: expert products that may share the launches of the first / the last product)
+static int mix_sink(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in, const DenseArgs* const* riders = nullptr) {
     const b2_layered_config& c = m->c;
     const b2_layer_desc& d = L.d;
     cudaStream_t st = e->stream;
@@ -1219,7 +1233,9 @@ static int mix_sink(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& 
     DenseArgs pj = {};
     pj.n_act = L.su_off; pj.n_act_end = L.su_off + Ko - od;       // the rows of a shared expert that rides along get their activation here
     if (in == m->hn) pj.x_rounded = m->hn_rounded;
+    m->rider = riders ? riders[0] : nullptr;
     if ((rc = dense(e, m, L.sk_proj, in, W, m->proj, Np, T, L.sk_bias, L.su_off >= 0 ? EPI_BIAS_PART_RELU2 : L.sk_bias ? EPI_BIAS : EPI_NONE, 1, &pj))) return rc;
+    if (m->rider) { if ((rc = dense_run(e, m, *std::exchange(m->rider, nullptr), 1))) return rc; }
     SinkAttnArgs a = {};
     a.proj = m->proj; a.ldp = Np; a.q_off = L.q_off; a.k_off = L.k_off; a.v_off = L.v_off;
     a.rot.cos = L.rot_cos; a.rot.sin = L.rot_sin; a.rot.rot_dims = d.rot_dims; a.unit_qk = (d.attn_flags & B2_ATTN_UNIT_QK) ? 1 : 0;
@@ -1245,7 +1261,9 @@ static int mix_sink(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& 
         e->launches += L.talk ? 3 : 2;
         if (a.conv_w && a.taps > 1 && T > 8) e->launches++;
     }
+    m->rider = riders ? riders[1] : nullptr;
     if ((rc = dense(e, m, L.attn_o, m->buf[1], Ko, m->oL, W, T, L.o_bias, L.o_bias ? EPI_BIAS : EPI_NONE, 1, &op))) return rc;
+    if (m->rider) { if ((rc = dense_run(e, m, *std::exchange(m->rider, nullptr), 1))) return rc; }
     if (d.mixer != B2_MIX_SINK_DELTA) return B2_OK;
     const int Hr = d.mm_heads, G = d.key_heads, kd = G * d.mm_dim, vd = Hr * d.mm_vdim;
     ConvArgs cv = {};
@@ -1305,13 +1323,19 @@ static int ff_glu(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r,
     return dense(e, m, L.glu_down, m->ff, ff, out, W, T);
 }
 
-// defer != nullptr: the weighted sum of the expert outputs is left to the caller's residual kernel (described in *defer)
-static int ff_moe(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in, float* out, MoeJoinArgs* defer) {
+// The two grouped products of a mixture, ready to launch, and what the residual kernel needs to add up their output.
+struct MoeJobs {
+    DenseGroups g, g2;
+    DenseArgs up, down;
+    MoeJoinArgs join;
+};
+// routing (or the step's plan), sorting, product descriptions; `j` must outlive the launches
+static int moe_prepare(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in, MoeJobs& j) {
     const b2_layer_desc& d = L.d;
     cudaStream_t st = e->stream;
     const int T = r.T, W = m->c.n_embd, slots = d.moe_experts + d.moe_identity, pairs = T * d.moe_top, ff = d.n_ff;
     int rc;
-    DenseGroups g = {};
+    DenseGroups& g = j.g;
     g.n_groups = d.moe_experts;
     const bool tiled = T > MOE_FEW_TOKENS, table = d.moe_route == B2_ROUTE_TABLE;
     // long prompts in the serving mode: 128-row tiles through the large tensor-core kernel
@@ -1351,30 +1375,36 @@ static int ff_moe(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r,
     // (experts by token id share one weight, which the down product's epilogue applies)
     const float* out_weight = d.moe_scale_input || table ? nullptr : m->moe_weight;
     if (d.moe_scale_input) g.row_scale = tiled ? m->moe_row_weight : m->moe_weight;
-    DenseArgs up = {};
     g.x_rows = tiled ? x_rows : tok; g.w_stride = (long)L.gate_up.N * W; g.x_total_rows = T;
-    up.groups = &g;
+    DenseArgs up = {};
+    up.groups = &j.g;
     up.p0 = (float)d.moe_limit; up.p1 = (float)d.moe_alpha;
     if (big) {                                     // the activations only feed the down maps: left rounded
         if (in == m->hn) up.x_rounded = m->hn_rounded;
         up.y_rounded = m->moe_hb;
     }
     const int act = d.moe_expert == B2_EXPERT_CLAMPED ? EPI_GLU_CLAMP : d.moe_expert == B2_EXPERT_RELU2 ? EPI_BIAS_RELU2 : EPI_GLU_SILU;
-    if ((rc = dense(e, m, L.gate_up, in, W, m->moe_h, ff, pairs, nullptr, act, 1, &up))) return rc;
-    DenseGroups g2 = g;
-    g2.x_rows = nullptr; g2.row_scale = nullptr; g2.w_stride = (long)W * ff; g2.x_total_rows = pairs;
+    j.up = dense_args(m, L.gate_up, in, W, m->moe_h, ff, pairs, nullptr, act, &up);
+    j.g2 = g;
+    j.g2.x_rows = nullptr; j.g2.row_scale = nullptr; j.g2.w_stride = (long)W * ff; j.g2.x_total_rows = pairs;
     DenseArgs dn = {};
-    dn.groups = &g2;
+    dn.groups = &j.g2;
     if (big) dn.x_rounded = m->moe_hb;
     if (table) dn.scale = 1.f / (float)d.moe_top;
-    if ((rc = dense(e, m, L.e_down, m->moe_h, ff, m->moe_y, W, pairs, nullptr, EPI_NONE, 1, &dn))) return rc;
-    if (defer) {
-        defer->sel = sel; defer->weight = out_weight; defer->pos = tiled ? pos : nullptr; defer->rows = m->moe_y; defer->h = in;
-        defer->n_experts = d.moe_experts; defer->top = d.moe_top;
-        return B2_OK;
-    }
-    StepProfiler sp(m, st, 7);
-    CK(moe_combine_launch(sel, out_weight, tiled ? pos : nullptr, m->moe_y, in, d.moe_experts, d.moe_top, W, T, out, st));
+    j.down = dense_args(m, L.e_down, m->moe_h, ff, m->moe_y, W, pairs, nullptr, EPI_NONE, &dn);
+    j.join.sel = sel; j.join.weight = out_weight; j.join.pos = tiled ? pos : nullptr; j.join.rows = m->moe_y; j.join.h = in;
+    j.join.n_experts = d.moe_experts; j.join.top = d.moe_top;
+    return B2_OK;
+}
+
+// defer != nullptr: the weighted sum of the expert outputs is left to the caller's residual kernel (described in *defer)
+static int ff_moe(b2_engine* e, LayeredModel* m, LyLayer& L, const RaggedDev& r, const float* in, float* out, MoeJoinArgs* defer) {
+    MoeJobs j;
+    int rc;
+    if ((rc = moe_prepare(e, m, L, r, in, j)) || (rc = dense_run(e, m, j.up, 1)) || (rc = dense_run(e, m, j.down, 1))) return rc;
+    if (defer) { *defer = j.join; return B2_OK; }
+    StepProfiler sp(m, e->stream, 7);
+    CK(moe_combine_launch(j.join.sel, j.join.weight, j.join.pos, m->moe_y, in, L.d.moe_experts, L.d.moe_top, m->c.n_embd, r.T, out, e->stream));
     e->launches++;
     return B2_OK;
 }
@@ -1439,6 +1469,7 @@ static int run_layers(b2_engine* e, LayeredModel* m, const RaggedDev& r) {
         return B2_OK;
     };
     m->hn_rounded = nullptr;
+    m->rider = nullptr;
     if (c.block_style == B2_BLOCK_HYPER_RMS) {
         // The embedding sits in copy 0. A sublayer's output waits (in m->oL / m->oR / the mixture's rows) until the next boundary:
         // one kernel writes it back into all copies, reads the next sublayer's input and norms it.
@@ -1543,8 +1574,18 @@ static int run_layers(b2_engine* e, LayeredModel* m, const RaggedDev& r) {
                 if ((rc = boundary())) return rc;
             }
             LyLayer& L = m->layers[li];
-            if ((rc = run_mixer(e, m, L, r, m->hn))) return rc;
             pj.a = m->oL;
+            if (one_norm && T <= MOE_FEW_TOKENS && L.d.mixer == B2_MIX_SINK_ATTN && L.d.n_ff > 0 && L.d.ff_kind == B2_FF_MOE && L.d.moe_route == B2_ROUTE_TABLE &&
+                (L.d.moe_shared_ff == 0 || L.su_off >= 0)) {
+                // few tokens, experts known beforehand: their two products share the launches of the mixer's first and last
+                MoeJobs jobs;
+                if ((rc = moe_prepare(e, m, L, r, ff_in, jobs))) return rc;
+                const DenseArgs* const riders[2] = {&jobs.up, &jobs.down};
+                if ((rc = mix_sink(e, m, L, r, m->hn, riders))) return rc;
+                pj_moe = jobs.join;
+                continue;
+            }
+            if ((rc = run_mixer(e, m, L, r, m->hn))) return rc;
             if (L.d.n_ff > 0) {
                 const bool moe = L.d.ff_kind == B2_FF_MOE;
                 if ((rc = run_ff(e, m, L, r, ff_in, m->oR, moe ? &pj_moe : nullptr))) return rc;

@@ -79,6 +79,9 @@ struct DenseArgs {
     const DenseGroups* groups = nullptr;            // grouped product (T = number of pair rows)
 };
 cudaError_t dense_launch(const DenseArgs& a, cudaStream_t s);
+// Few-token steps: a plain product and an independent one over (token, choice) pairs in ONE launch (dense_pairs: the two qualify).
+bool dense_pairs(const DenseArgs& a, const DenseArgs& b);
+cudaError_t dense_pair_launch(const DenseArgs& a, const DenseArgs& b, cudaStream_t s);
 bool dense_takes_rounded(const DenseArgs& a);          // dense_launch takes the kernel that reads rounded inputs
 
 // ---------------------------------------------------------------- mixers and norms (mixers.cu)
