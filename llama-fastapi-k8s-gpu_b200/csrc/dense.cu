@@ -38,7 +38,7 @@ struct DenseDev {
 // The rows [t0, t1) this CTA computes and the operands they use. false: nothing to do.
 template <typename TW>
 __device__ __forceinline__ bool dense_tile(const DenseDev& a, int rows_per_cta, const float*& x, const TW*& w, float*& y, const float*& aux,
-                                           int& t0, int& t1, int by, int bz) {
+                                           int& t0, int& t1, unsigned by, unsigned bz) {
     x = a.x; w = reinterpret_cast<const TW*>(a.w); y = a.y; aux = a.aux;
     if (a.grouped == 0) {
         const long b = bz;
@@ -119,7 +119,7 @@ __device__ __forceinline__ void epi_store2(const DenseDev& a, float* y, const fl
 // over k in an order that depends on K alone.
 constexpr int ROWS_MAX_T = 8;
 template <typename TW, int TT, int R>
-__device__ __forceinline__ void dense_rows_cta(const DenseDev& a, int bx, int by, int bz) {
+__device__ __forceinline__ void dense_rows_cta(const DenseDev& a, unsigned bx, unsigned by, unsigned bz) {
     constexpr int U = 4 / R;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int N = a.N, K = a.K, ldx = a.ldx;
@@ -217,10 +217,10 @@ __global__ void __launch_bounds__(256) dense_rows_kernel(DenseDev a) {
 }
 // two independent products in one launch: the CTAs of a, then those of b (grouped pairs, `nb` CTAs each)
 template <typename TW, int TT, int R>
-__global__ void __launch_bounds__(256) dense_rows_pair_kernel(DenseDev a, DenseDev b, int na, int nb) {
+__global__ void __launch_bounds__(256) dense_rows_pair_kernel(DenseDev a, DenseDev b, unsigned na, unsigned nb) {
     griddep_launch();
     griddep_wait();
-    if ((int)blockIdx.x < na) dense_rows_cta<TW, TT, R>(a, blockIdx.x, 0, 0);
+    if (blockIdx.x < na) dense_rows_cta<TW, TT, R>(a, blockIdx.x, 0, 0);
     else dense_rows_cta<TW, 1, 1>(b, (blockIdx.x - na) % nb, (blockIdx.x - na) / nb, 0);
 }
 
@@ -499,7 +499,7 @@ bool dense_pairs(const DenseArgs& a, const DenseArgs& b) {
 }
 template <typename TW>
 static cudaError_t launch_rows_pair(const DenseDev& a, const DenseDev& b, cudaStream_t s) {
-    const int per = a.T == 1 ? 8 : a.T == 2 ? 16 : 32, na = (a.N + per - 1) / per, nb = (b.N + 7) / 8;      // rows per CTA as in launch_rows
+    const unsigned per = a.T == 1 ? 8 : a.T == 2 ? 16 : 32, na = (a.N + per - 1) / per, nb = (b.N + 7) / 8;      // rows per CTA as in launch_rows
     const dim3 grid(na + nb * b.T), block(256);
     if (a.T == 1) return launch_chain(dense_rows_pair_kernel<TW, 1, 1>, grid, block, 0, s, a, b, na, nb);
     if (a.T == 2) return launch_chain(dense_rows_pair_kernel<TW, 2, 2>, grid, block, 0, s, a, b, na, nb);
